@@ -1,4 +1,4 @@
-"""ctypes binding of the C ABI declared in ``include/tilert_b200.h``.
+"""ctypes binding of the C ABIs declared in ``include/*.h`` (one header per native library).
 
 The prototypes are read from the header itself, so the Python side cannot drift from the
 declarations: every function the header declares must be exported by the library, and is
@@ -11,7 +11,11 @@ import ctypes
 import re
 from pathlib import Path
 
-HEADER = Path(__file__).resolve().parent.parent / "include" / "tilert_b200.h"
+def header_path(name: str) -> Path:
+    return Path(__file__).resolve().parent.parent / "include" / name
+
+
+HEADER = header_path("tilert_b200.h")
 
 _SCALARS = {
     "int": ctypes.c_int,
@@ -44,9 +48,9 @@ def parse_header(path: Path = HEADER) -> dict[str, tuple[object, list[object]]]:
     return protos
 
 
-def bind(lib_path: Path) -> ctypes.CDLL:
-    lib = ctypes.CDLL(str(lib_path), mode=ctypes.RTLD_GLOBAL)
-    for name, (restype, argtypes) in parse_header().items():
+def bind(lib_path: Path, header: Path = HEADER, exported_globally: bool = True) -> ctypes.CDLL:
+    lib = ctypes.CDLL(str(lib_path), mode=ctypes.RTLD_GLOBAL if exported_globally else ctypes.RTLD_LOCAL)
+    for name, (restype, argtypes) in parse_header(header).items():
         fn = getattr(lib, name)  # AttributeError here = header/library mismatch
         fn.restype = restype
         fn.argtypes = argtypes

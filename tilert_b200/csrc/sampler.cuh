@@ -13,7 +13,7 @@
 #pragma once
 
 #include "common.cuh"
-#include "indexer.cuh"
+#include "topk_radix.cuh"
 
 namespace tb {
 

@@ -1,0 +1,521 @@
+// Grouped-query attention over a ring of cached keys and values.
+//
+// A cache holds, per key/value head, `ring` rows; position p lives in row p mod ring.  A query at position i sees
+// the positions j with 0 <= i - j < window (window 0: every j <= i); the ring has to hold the window of the oldest
+// query of a launch together with every position of the launch.  Rows are padded to 16 elements with zeros.
+//
+// Queries and keys are RMS-normalised over their whole projection (all heads at once) before they are split into
+// heads; values can be mixed with the values an earlier layer had for the same token.  Both happen here:
+//   qkv_rows_kernel          a portion of tokens: normalised queries out, keys and values into the ring
+//   attn_prefill_kernel      a portion of tokens, bf16 tensor-core tiles with an online softmax
+//   attn_rows_kernel<T, true>   one token: the preparation, the cache write and the attention in one launch, the
+//                            keys split over CTAs, the last CTA of a head block merging the parts
+//   attn_rows_kernel<T, false>  any number of prepared query rows, f32 arithmetic (the exact mode)
+// Scores, softmax and sums are f32 throughout.
+#pragma once
+
+#include "act.cuh"
+
+namespace tb {
+
+enum ValueMix : int { VMIX_NONE = 0, VMIX_FIRST = 1, VMIX_BLEND = 2 };
+
+struct QkvShape {
+  int heads, kv_heads, dim, vdim;
+  int dimp, vdimp;       // padded to 16
+  int ring;              // cache rows per head
+  int window;            // 0: no window
+};
+
+struct QkvPrep {
+  const float* qkv;      // [rows, ld]: queries, keys, values of one token
+  long long ld;
+  const float* q_gain;   // [heads * dim]
+  const float* k_gain;   // [kv_heads * dim]
+  float eps;
+  int v_mode;
+  const float* lambda;   // one value (VMIX_BLEND)
+  float* v_first;        // [rows, kv_heads * vdim] written (VMIX_FIRST) or read (VMIX_BLEND)
+};
+
+// Value element e (over all heads) of row `t`, after mixing; VMIX_FIRST also leaves it for the later layers.
+__device__ __forceinline__ float mixed_value(const QkvPrep& p, const QkvShape& s, int t, int e, bool store_first) {
+  const int nq = s.heads * s.dim, nk = s.kv_heads * s.dim, nv = s.kv_heads * s.vdim;
+  const float v = p.qkv[t * p.ld + nq + nk + e];
+  if (p.v_mode == VMIX_FIRST && store_first) p.v_first[static_cast<long long>(t) * nv + e] = v;
+  if (p.v_mode == VMIX_BLEND) {
+    const float l = *p.lambda;
+    return (1.f - l) * v + l * p.v_first[static_cast<long long>(t) * nv + e];
+  }
+  return v;
+}
+
+__device__ __forceinline__ float rinv_of(float sum, int n, float eps) { return 1.f / sqrtf(sum / static_cast<float>(n) + eps); }
+
+// ------------------------------------------------------------------ a portion of tokens: prepare
+struct QkvRowsParams {
+  QkvShape s;
+  QkvPrep p;
+  const int* pos;        // position of row 0
+  void* q;               // [rows, heads, dimp] normalised queries (padding left as it is: zero)
+  void* k_cache;         // [kv_heads, ring, dimp]
+  void* v_cache;         // [kv_heads, ring, vdimp]
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) qkv_rows_kernel(const QkvRowsParams a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[32];
+  const QkvShape& s = a.s;
+  const int t = blockIdx.x;
+  const float* row = a.p.qkv + t * a.p.ld;
+  const int nq = s.heads * s.dim, nk = s.kv_heads * s.dim, nv = s.kv_heads * s.vdim;
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x; i < nq; i += 256) sq += row[i] * row[i];
+  for (int i = threadIdx.x; i < nk; i += 256) sk += row[nq + i] * row[nq + i];
+  const float rq = rinv_of(cta_sum(sq, red), nq, a.p.eps), rk = rinv_of(cta_sum(sk, red), nk, a.p.eps);
+  const long long slot = (*a.pos + t) % s.ring;
+  T* q = reinterpret_cast<T*>(a.q) + static_cast<long long>(t) * s.heads * s.dimp;
+  T* kc = reinterpret_cast<T*>(a.k_cache);
+  T* vc = reinterpret_cast<T*>(a.v_cache);
+  for (int i = threadIdx.x; i < nq; i += 256) {
+    const int h = i / s.dim;
+    act_st(q + h * s.dimp + i - h * s.dim, row[i] * rq * a.p.q_gain[i]);
+  }
+  for (int i = threadIdx.x; i < nk; i += 256) {
+    const int g = i / s.dim;
+    act_st(kc + (static_cast<long long>(g) * s.ring + slot) * s.dimp + i - g * s.dim, row[nq + i] * rk * a.p.k_gain[i]);
+  }
+  for (int i = threadIdx.x; i < nv; i += 256) {
+    const int g = i / s.vdim;
+    act_st(vc + (static_cast<long long>(g) * s.ring + slot) * s.vdimp + i - g * s.vdim, mixed_value(a.p, s, t, i, true));
+  }
+}
+
+// ------------------------------------------------------------------ query rows against a range of keys, f32
+constexpr int kAttnThreads = 256;
+constexpr int kAttnHeads = 4;    // query heads per CTA
+constexpr int kAttnChunk = 128;  // keys per softmax step
+
+struct AttnRowsParams {
+  QkvShape s;
+  QkvPrep p;             // FUSED
+  const int* pos;        // position of row 0
+  const void* q;         // !FUSED: [rows, heads, dimp]
+  void* k_cache;
+  void* v_cache;
+  float scale;
+  int n_splits;
+  float* part;           // [heads, n_splits, vdimp] and, behind it, [heads, n_splits, 2] (max, sum)
+  unsigned* counter;     // [head blocks], zero between launches
+  void* out;             // [rows, ldo], element type float (FUSED) or T
+  long long ldo;
+};
+
+__host__ __device__ inline size_t attn_rows_smem(int dimp, int vdimp) {
+  return (kAttnHeads * dimp + kAttnHeads * kAttnChunk + kAttnThreads * kAttnHeads * 8) * sizeof(float);
+}
+
+template <typename T, bool FUSED>
+__global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsParams a) {
+  extern __shared__ __align__(16) float smem[];
+  __shared__ float red[32];
+  __shared__ float s_m[kAttnHeads], s_l[kAttnHeads], s_corr[kAttnHeads];
+  __shared__ int s_last;
+  pdl_launch_dependents();
+  pdl_wait();
+  const QkvShape& s = a.s;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int group = s.heads / s.kv_heads, n_hb = (group + kAttnHeads - 1) / kAttnHeads;
+  const int split = blockIdx.x, g = blockIdx.y / n_hb, hb = blockIdx.y - g * n_hb, t = blockIdx.z;
+  const int h0 = g * group + hb * kAttnHeads;
+  const int nh = min(kAttnHeads, group - hb * kAttnHeads);
+  const int pos = *a.pos + t;
+  float* qs = smem;                               // [kAttnHeads][dimp], scaled
+  float* sc = qs + kAttnHeads * s.dimp;           // [kAttnHeads][kAttnChunk]
+  float* red2 = sc + kAttnHeads * kAttnChunk;     // [threads][kAttnHeads * 8]
+  const int first = s.window > 0 ? max(0, pos - s.window + 1) : 0;
+  const int n = pos + 1 - first;
+  const int per = (n + a.n_splits - 1) / a.n_splits;
+  const int lo = min(first + split * per, pos + 1), hi = min(lo + per, pos + 1);
+  T* kc = reinterpret_cast<T*>(a.k_cache) + static_cast<long long>(g) * s.ring * s.dimp;
+  T* vc = reinterpret_cast<T*>(a.v_cache) + static_cast<long long>(g) * s.ring * s.vdimp;
+
+  if (FUSED) {
+    const int nq = s.heads * s.dim, nk = s.kv_heads * s.dim;
+    const float* row = a.p.qkv;
+    float sq = 0.f, sk = 0.f;
+    for (int i = tid; i < nq; i += kAttnThreads) sq += row[i] * row[i];
+    for (int i = tid; i < nk; i += kAttnThreads) sk += row[nq + i] * row[nq + i];
+    const float rq = rinv_of(cta_sum(sq, red), nq, a.p.eps), rk = rinv_of(cta_sum(sk, red), nk, a.p.eps);
+    for (int i = tid; i < kAttnHeads * s.dimp; i += kAttnThreads) {
+      const int h = i / s.dimp, d = i - h * s.dimp;
+      const int e = (h0 + h) * s.dim + d;
+      qs[i] = h < nh && d < s.dim ? row[e] * rq * a.p.q_gain[e] * a.scale : 0.f;
+    }
+    if (lo < hi && hi == pos + 1) {  // the CTAs whose range holds the current position write (the same) cache row
+      const long long slot = pos % s.ring;
+      for (int d = tid; d < s.dim; d += kAttnThreads) {
+        const int e = g * s.dim + d;
+        act_st(kc + slot * s.dimp + d, row[nq + e] * rk * a.p.k_gain[e]);
+      }
+      for (int d = tid; d < s.vdim; d += kAttnThreads)
+        act_st(vc + slot * s.vdimp + d, mixed_value(a.p, s, 0, g * s.vdim + d, true));
+    }
+  } else {
+    const T* q = reinterpret_cast<const T*>(a.q) + (static_cast<long long>(t) * s.heads + h0) * s.dimp;
+    for (int i = tid; i < kAttnHeads * s.dimp; i += kAttnThreads) qs[i] = i / s.dimp < nh ? act_ld(q + i) * a.scale : 0.f;
+  }
+  if (tid < kAttnHeads) {
+    s_m[tid] = -INFINITY;
+    s_l[tid] = 0.f;
+  }
+  __syncthreads();  // queries staged, the current cache row visible to this CTA
+
+  const int n_vc = s.vdimp / 8;                    // value pieces; thread = (key lane, piece)
+  const int key_lanes = kAttnThreads / n_vc;
+  const int kl = tid / n_vc, vp = tid - kl * n_vc;
+  const bool v_active = kl < key_lanes;
+  float acc[kAttnHeads][8];
+#pragma unroll
+  for (int h = 0; h < kAttnHeads; ++h)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) acc[h][j] = 0.f;
+
+  // the keys of a launch lie in fewer than `ring` consecutive positions, so one subtraction wraps a row index
+  for (int c0 = lo; c0 < hi; c0 += kAttnChunk) {
+    const int cn = min(kAttnChunk, hi - c0), slot0 = c0 % s.ring;
+    // scores: eight lanes per key, four keys per warp and step
+    for (int k0 = warp * 4; k0 < kAttnChunk; k0 += kAttnThreads / 8) {
+      const int key = k0 + (lane >> 3);
+      float d[kAttnHeads];
+#pragma unroll
+      for (int h = 0; h < kAttnHeads; ++h) d[h] = 0.f;
+      if (key < cn) {
+        const int slot = slot0 + key - (slot0 + key >= s.ring ? s.ring : 0);
+        const T* kr = kc + static_cast<long long>(slot) * s.dimp;
+        for (int c = lane & 7; c < s.dimp / 8; c += 8) {
+          float f[8];
+          act_ld8(kr + c * 8, f);
+#pragma unroll
+          for (int h = 0; h < kAttnHeads; ++h) {
+            const float4 q0 = *reinterpret_cast<const float4*>(qs + h * s.dimp + c * 8);
+            const float4 q1 = *reinterpret_cast<const float4*>(qs + h * s.dimp + c * 8 + 4);
+            d[h] += f[0] * q0.x + f[1] * q0.y + f[2] * q0.z + f[3] * q0.w + f[4] * q1.x + f[5] * q1.y + f[6] * q1.z + f[7] * q1.w;
+          }
+        }
+      }
+#pragma unroll
+      for (int h = 0; h < kAttnHeads; ++h) {
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) d[h] += __shfl_xor_sync(0xffffffffu, d[h], o);
+        if ((lane & 7) == 0) sc[h * kAttnChunk + key] = key < cn ? d[h] : -INFINITY;
+      }
+    }
+    __syncthreads();
+    if (warp < kAttnHeads) {
+      float m = -INFINITY;
+      for (int i = lane; i < kAttnChunk; i += 32) m = fmaxf(m, sc[warp * kAttnChunk + i]);
+      m = fmaxf(warp_max(m), s_m[warp]);
+      float l = 0.f;
+      for (int i = lane; i < kAttnChunk; i += 32) {
+        const float e = expf(sc[warp * kAttnChunk + i] - m);
+        sc[warp * kAttnChunk + i] = e;
+        l += e;
+      }
+      l = warp_sum(l);
+      if (lane == 0) {
+        const float corr = expf(s_m[warp] - m);
+        s_corr[warp] = corr;
+        s_l[warp] = s_l[warp] * corr + l;
+        s_m[warp] = m;
+      }
+    }
+    __syncthreads();
+    if (v_active) {
+#pragma unroll
+      for (int h = 0; h < kAttnHeads; ++h)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[h][j] *= s_corr[h];
+      for (int key = kl; key < cn; key += key_lanes) {
+        float f[8];
+        const int slot = slot0 + key - (slot0 + key >= s.ring ? s.ring : 0);
+        act_ld8(vc + static_cast<long long>(slot) * s.vdimp + vp * 8, f);
+#pragma unroll
+        for (int h = 0; h < kAttnHeads; ++h) {
+          const float w = sc[h * kAttnChunk + key];
+#pragma unroll
+          for (int j = 0; j < 8; ++j) acc[h][j] += w * f[j];
+        }
+      }
+    }
+    __syncthreads();
+  }
+
+  // sum over the key lanes: red2[kl][h][vdimp]
+  if (v_active) {
+#pragma unroll
+    for (int h = 0; h < kAttnHeads; ++h)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) red2[(kl * kAttnHeads + h) * s.vdimp + vp * 8 + j] = acc[h][j];
+  }
+  __syncthreads();
+  const bool whole = a.n_splits == 1;
+  float* ml = a.part + static_cast<long long>(s.heads) * a.n_splits * s.vdimp;
+  for (int i = tid; i < nh * s.vdimp; i += kAttnThreads) {
+    const int h = i / s.vdimp, v = i - h * s.vdimp;
+    float o = 0.f;
+    for (int k = 0; k < key_lanes; ++k) o += red2[(k * kAttnHeads + h) * s.vdimp + v];
+    if (!whole) {
+      a.part[(static_cast<long long>(h0 + h) * a.n_splits + split) * s.vdimp + v] = o;
+    } else if (v < s.vdim) {
+      const long long dst = t * a.ldo + (h0 + h) * s.vdim + v;
+      if (FUSED)
+        reinterpret_cast<float*>(a.out)[dst] = o / s_l[h];
+      else
+        act_st(reinterpret_cast<T*>(a.out) + dst, o / s_l[h]);
+    }
+  }
+  if (whole) return;
+  if (tid < nh) {
+    ml[((h0 + tid) * a.n_splits + split) * 2] = s_m[tid];
+    ml[((h0 + tid) * a.n_splits + split) * 2 + 1] = s_l[tid];
+  }
+  // merge by the CTA that finishes its head block last (no CTA waits for another)
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) {
+    const unsigned prev = atomicAdd(a.counter + blockIdx.y, 1u);
+    s_last = prev == static_cast<unsigned>(a.n_splits) - 1u;
+    if (s_last) a.counter[blockIdx.y] = 0u;
+  }
+  __syncthreads();
+  if (!s_last) return;
+  __threadfence();
+  for (int i = tid; i < nh * s.vdim; i += kAttnThreads) {
+    const int h = i / s.vdim, v = i - h * s.vdim;
+    const float* mh = ml + (h0 + h) * a.n_splits * 2;
+    float m = -INFINITY;
+    for (int k = 0; k < a.n_splits; ++k) m = fmaxf(m, __ldcg(mh + 2 * k));
+    float o = 0.f, l = 0.f;
+    for (int k = 0; k < a.n_splits; ++k) {
+      const float c = expf(__ldcg(mh + 2 * k) - m);  // an empty part has max -inf: weight 0
+      l += c * __ldcg(mh + 2 * k + 1);
+      o += c * __ldcg(a.part + (static_cast<long long>(h0 + h) * a.n_splits + k) * s.vdimp + v);
+    }
+    const long long dst = t * a.ldo + (h0 + h) * s.vdim + v;
+    if (FUSED)
+      reinterpret_cast<float*>(a.out)[dst] = o / l;
+    else
+      act_st(reinterpret_cast<T*>(a.out) + dst, o / l);
+  }
+}
+
+// ------------------------------------------------------------------ a portion of tokens, bf16 tensor-core tiles
+// 64 rows per CTA = (tokens x query heads of one key/value head), so the heads of a group share the key tiles.
+// 64 keys per tile, two tiles in flight (cp.async); four warps of 16 rows; online softmax in registers.
+constexpr int kFaRows = 64, kFaKeys = 64, kFaThreads = 128;
+constexpr int kFaMaxHeads = 16;  // query heads of a group per CTA
+
+struct AttnPrefillParams {
+  QkvShape s;
+  const int* pos;        // position of row 0
+  int rows;
+  const __nv_bfloat16* q;        // [rows, heads, dimp]
+  const __nv_bfloat16* k_cache;  // [kv_heads, ring, dimp]
+  const __nv_bfloat16* v_cache;  // [kv_heads, ring, vdimp]
+  float scale;
+  __nv_bfloat16* out;    // [rows, ldo]
+  long long ldo;
+};
+
+__host__ __device__ inline size_t attn_prefill_smem(int dimp, int vdimp) {
+  return (static_cast<size_t>(kFaRows + 2 * kFaKeys) * (dimp + 8) + 2 * kFaKeys * (vdimp + 8)) * 2;
+}
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// DV16: value tiles of 16 columns the accumulator has room for (vdimp <= 16 * DV16)
+template <int DV16>
+__global__ void __launch_bounds__(kFaThreads) attn_prefill_kernel(const AttnPrefillParams a) {
+  extern __shared__ __align__(16) __nv_bfloat16 fsm[];
+  pdl_launch_dependents();
+  pdl_wait();
+  const QkvShape& s = a.s;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int group = s.heads / s.kv_heads;
+  const int hpb = min(group, kFaMaxHeads), n_hb = (group + hpb - 1) / hpb;
+  const int tpb = kFaRows / hpb;  // tokens per CTA
+  const int g = blockIdx.y / n_hb, hb = blockIdx.y - g * n_hb;
+  const int h0 = g * group + hb * hpb, nh = min(hpb, group - hb * hpb);
+  const int t0 = (gridDim.x - 1 - blockIdx.x) * tpb;  // the longest ranges first
+  const int nt = min(tpb, a.rows - t0);
+  const int pos0 = *a.pos;
+  const int qp = s.dimp + 8, vpitch = s.vdimp + 8;
+  __nv_bfloat16* qs = fsm;
+  __nv_bfloat16* ks = qs + kFaRows * qp;
+  __nv_bfloat16* vs = ks + 2 * kFaKeys * qp;
+  const __nv_bfloat16* kc = a.k_cache + static_cast<long long>(g) * s.ring * s.dimp;
+  const __nv_bfloat16* vc = a.v_cache + static_cast<long long>(g) * s.ring * s.vdimp;
+  const int lo = s.window > 0 ? max(0, pos0 + t0 - s.window + 1) : 0, hi = pos0 + t0 + nt;  // keys any row sees
+
+  const int dch = s.dimp / 8, vch = s.vdimp / 8;
+  for (int i = tid; i < kFaRows * dch; i += kFaThreads) {
+    const int r = i / dch, c = i - r * dch;
+    const int tt = r / hpb, h = r - tt * hpb;
+    const bool ok = tt < nt && h < nh;
+    const long long row = ok ? static_cast<long long>(t0 + tt) * s.heads + h0 + h : 0;
+    cp_async16(qs + r * qp + c * 8, a.q + row * s.dimp + c * 8, ok);
+  }
+  auto load_tile = [&](int k0, int buf) {
+    __nv_bfloat16* kd = ks + buf * kFaKeys * qp;
+    __nv_bfloat16* vd = vs + buf * kFaKeys * vpitch;
+    const int slot0 = k0 % s.ring;
+    for (int i = tid; i < kFaKeys * dch; i += kFaThreads) {
+      const int r = i / dch, c = i - r * dch;
+      const bool ok = k0 + r < hi;
+      const long long slot = ok ? slot0 + r - (slot0 + r >= s.ring ? s.ring : 0) : 0;
+      cp_async16(kd + r * qp + c * 8, kc + slot * s.dimp + c * 8, ok);
+    }
+    for (int i = tid; i < kFaKeys * vch; i += kFaThreads) {
+      const int r = i / vch, c = i - r * vch;
+      const bool ok = k0 + r < hi;
+      const long long slot = ok ? slot0 + r - (slot0 + r >= s.ring ? s.ring : 0) : 0;
+      cp_async16(vd + r * vpitch + c * 8, vc + slot * s.vdimp + c * 8, ok);
+    }
+    cp_async_commit();
+  };
+  load_tile(lo, 0);
+
+  float o[DV16 * 2][4];
+#pragma unroll
+  for (int i = 0; i < DV16 * 2; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  // this thread's two rows (lane / 4 and + 8 inside the warp's 16)
+  int qpos[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = warp * 16 + (lane >> 2) + i * 8, tt = r / hpb;
+    qpos[i] = tt < nt ? pos0 + t0 + tt : -1;  // a row without a token sees nothing
+  }
+  const int win = s.window > 0 ? s.window : 0x7fffffff;
+  const int n_tiles = (hi - lo + kFaKeys - 1) / kFaKeys;
+  for (int tile = 0; tile < n_tiles; ++tile) {
+    const int k0 = lo + tile * kFaKeys, buf = tile & 1;
+    if (tile + 1 < n_tiles) {
+      load_tile(k0 + kFaKeys, buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const __nv_bfloat16* kt = ks + buf * kFaKeys * qp;
+    const __nv_bfloat16* vt = vs + buf * kFaKeys * vpitch;
+    float sacc[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) sacc[i][j] = 0.f;
+    for (int kk = 0; kk < s.dimp / 16; ++kk) {
+      uint32_t qa[4];
+      ldmatrix_x4(qa, qs + (warp * 16 + (lane & 15)) * qp + kk * 16 + (lane >> 4) * 8);
+#pragma unroll
+      for (int nb = 0; nb < 4; ++nb) {
+        uint32_t kb[4];  // two tiles of eight keys: (k 0-7, k 8-15) each
+        ldmatrix_x4(kb, kt + (nb * 16 + (lane & 7) + (lane >> 4) * 8) * qp + kk * 16 + ((lane >> 3) & 1) * 8);
+        const uint32_t b0[2] = {kb[0], kb[1]}, b1[2] = {kb[2], kb[3]};
+        mma_bf16_16816(sacc[nb * 2], qa, b0);
+        mma_bf16_16816(sacc[nb * 2 + 1], qa, b1);
+      }
+    }
+    float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int nt8 = 0; nt8 < 8; ++nt8)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int kpos = k0 + nt8 * 8 + (lane & 3) * 2 + (j & 1), i = j >> 1;
+        const bool ok = kpos <= qpos[i] && qpos[i] - kpos < win;
+        sacc[nt8][j] = ok ? sacc[nt8][j] * a.scale : -INFINITY;
+        mx[i] = fmaxf(mx[i], sacc[nt8][j]);
+      }
+    float corr[2], msafe[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+      const float mn = fmaxf(m[i], mx[i]);
+      msafe[i] = mn == -INFINITY ? 0.f : mn;
+      corr[i] = __expf(m[i] - msafe[i]);
+      m[i] = mn;
+      l[i] *= corr[i];
+    }
+#pragma unroll
+    for (int i = 0; i < DV16 * 2; ++i) {
+      o[i][0] *= corr[0];
+      o[i][1] *= corr[0];
+      o[i][2] *= corr[1];
+      o[i][3] *= corr[1];
+    }
+    uint32_t pa[4][4];
+#pragma unroll
+    for (int nb = 0; nb < 4; ++nb) {
+      float e[8];
+#pragma unroll
+      for (int q = 0; q < 2; ++q)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float v = __expf(sacc[nb * 2 + q][j] - msafe[j >> 1]);
+          e[q * 4 + j] = v;
+          l[j >> 1] += v;
+        }
+      pa[nb][0] = pack_bf16x2(e[0], e[1]);
+      pa[nb][1] = pack_bf16x2(e[2], e[3]);
+      pa[nb][2] = pack_bf16x2(e[4], e[5]);
+      pa[nb][3] = pack_bf16x2(e[6], e[7]);
+    }
+#pragma unroll
+    for (int vb = 0; vb < DV16; ++vb) {
+      if (vb * 16 < s.vdimp) {
+#pragma unroll
+        for (int nb = 0; nb < 4; ++nb) {
+          uint32_t bv[4];  // keys 0-7 / 8-15 of columns 0-7, then of columns 8-15
+          ldmatrix_x4_trans(bv, vt + (nb * 16 + (lane & 15)) * vpitch + vb * 16 + (lane >> 4) * 8);
+          const uint32_t b0[2] = {bv[0], bv[1]}, b1[2] = {bv[2], bv[3]};
+          mma_bf16_16816(o[vb * 2], pa[nb], b0);
+          mma_bf16_16816(o[vb * 2 + 1], pa[nb], b1);
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
+    l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
+    const int r = warp * 16 + (lane >> 2) + i * 8, tt = r / hpb, h = r - tt * hpb;
+    if (tt >= nt || h >= nh) continue;
+    const float inv = 1.f / l[i];
+    __nv_bfloat16* dst = a.out + static_cast<long long>(t0 + tt) * a.ldo + (h0 + h) * s.vdim;
+    const bool pairs = (s.vdim & 1) == 0;
+#pragma unroll
+    for (int vb = 0; vb < DV16 * 2; ++vb) {
+      const int c = vb * 8 + (lane & 3) * 2;
+      if (pairs) {
+        if (c < s.vdim) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(o[vb][i * 2] * inv, o[vb][i * 2 + 1] * inv);
+      } else {
+        if (c < s.vdim) dst[c] = f2bf(o[vb][i * 2] * inv);
+        if (c + 1 < s.vdim) dst[c + 1] = f2bf(o[vb][i * 2 + 1] * inv);
+      }
+    }
+  }
+}
+
+}  // namespace tb

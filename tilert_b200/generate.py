@@ -4,6 +4,8 @@ this backend.  No checkpoint or tokenizer ships with the repository, so the runn
 ``prompt_tokens=`` path, generator.py:160,195).
 
     python -m tilert_b200.generate --model toy --use-random-weights --max-new-tokens 32 [--with-mtp]
+    python -m tilert_b200.generate --model ralasun --use-random-weights [--dtype float32]
+    python -m tilert_b200.generate --model-weights-dir DIR      # the family is chosen by DIR/config.json
 """
 
 from __future__ import annotations
@@ -13,14 +15,18 @@ import statistics
 
 import torch
 
+from tilert_b200.models import registry
+
 
 def parse_args():
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
-    ap.add_argument("--model", default="toy", choices=["toy", "deepseek_v3_2"],
-                    help="toy: the 2-layer test model; deepseek_v3_2: the full shape with --layers layers")
+    ap.add_argument("--model", default="toy", choices=registry.presets(),
+                    help="toy: the 2-layer test model; deepseek_v3_2: the full shape with --layers layers; ralasun: a small "
+                         "model of that design")
+    ap.add_argument("--dtype", default="bfloat16", help="activation type of a family that runs in more than one")
     ap.add_argument("--layers", type=int, default=2, help="decoder layers of the full-shape model (61 in the real one)")
     ap.add_argument("--use-random-weights", action="store_true")
-    ap.add_argument("--model-weights-dir", default=None, help="directory written by python -m tilert_b200.convert")
+    ap.add_argument("--model-weights-dir", default=None, help="checkpoint directory: config.json and *.safetensors")
     ap.add_argument("--with-mtp", action="store_true")
     ap.add_argument("--max-new-tokens", type=int, default=32)
     ap.add_argument("--prompt-len", type=int, default=16)
@@ -35,32 +41,24 @@ def parse_args():
 def main() -> None:
     args = parse_args()
     import tilert_b200
-    from tilert_b200.models.deepseek_v3_2.generator import DSAv32Generator
-    from tilert_b200.models.deepseek_v3_2.model_args import ModelArgs, toy_model_args
-    from dataclasses import replace
 
     if not torch.cuda.is_available():
         raise SystemExit("tilert_b200.generate needs a CUDA device (sm_100a); there is no CPU path")
-    tilert_b200.load_backend("deepseek_v3_2")
-    tilert_b200.tilert_init(0)
-    if args.model == "toy":
-        margs = replace(toy_model_args(), max_seq_len=args.max_seq_len)
-    else:
-        margs = replace(ModelArgs(), n_layers=args.layers, n_dense_layers=min(3, args.layers - 1), max_seq_len=args.max_seq_len)
-    gen = DSAv32Generator(margs, max_new_tokens=args.max_new_tokens, with_mtp=args.with_mtp, sampling_seed=args.seed,
-                          max_seq_len=args.max_seq_len)
-    if args.use_random_weights or args.model_weights_dir is None:
-        gen.init_random_weights(args.seed)
-    else:
-        from tilert_b200 import convert
-
-        gen.from_state_dict(convert.load_state_dict(args.model_weights_dir))
+    weights_dir = None if args.use_random_weights else args.model_weights_dir
+    family = registry.family_of_preset(args.model) if weights_dir is None else registry.family_of_dir(weights_dir)
+    if args.dtype not in family.dtypes:
+        raise SystemExit(f"{family.name} runs in {', '.join(family.dtypes)}, not in {args.dtype}")
+    if args.with_mtp and family.name != "deepseek_v3_2":
+        raise SystemExit(f"{family.name} has no multi-token prediction layer")
+    tilert_b200.load_backend(family.name)
+    tilert_b200.tilert_init(0, family.name)
+    gen = family.generator(weights_dir, args)
     if args.temperature > 0:
         gen.update_sampling_config(args.temperature, args.top_p, args.top_k, args.top_p < 1.0)
     g = torch.Generator().manual_seed(args.seed + 1)
-    prompt = torch.randint(0, margs.vocab_size, (args.prompt_len,), generator=g).tolist()
+    prompt = torch.randint(0, gen.vocab_size(), (args.prompt_len,), generator=g).tolist()
     text, times, accepted, plen = gen.generate("", print_log=True, prompt_tokens=prompt)
-    decode = times[plen:] if not args.with_mtp else times[-len(accepted):]
+    decode = times[-len(accepted):] if args.with_mtp else times[gen.prompt_steps(plen):]
     if decode:
         per_step = statistics.median(decode)
         toks = (sum(accepted) / len(accepted)) if accepted else 1.0

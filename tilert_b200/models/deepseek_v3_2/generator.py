@@ -1,8 +1,6 @@
 """Single-sequence generation on top of ``ShowHandsDSALayer``: the reference's ``DSAv32Generator``
 (tilert/models/deepseek_v3_2/generator.py:45-540) -- token-by-token prefill then decode, with or without
-multi-token prediction, per-token wall-clock times, and the synthetic-workload entry ``prompt_tokens=``.
-A tokenizer is optional (none ships with this repository): without one, prompts are token id lists and the
-returned text is the space-joined ids."""
+multi-token prediction, per-token wall-clock times, and the synthetic-workload entry ``prompt_tokens=``."""
 
 from __future__ import annotations
 
@@ -10,13 +8,14 @@ import time
 
 import torch
 
+from ..generator import SequenceGenerator
 from .end2end import ShowHandsDSALayer
 from .model_args import ModelArgs
 from .mtp import N_TOKENS
 from .temp_var_indices import Idx
 
 
-class DSAv32Generator:
+class DSAv32Generator(SequenceGenerator):
     def __init__(self, model_args: ModelArgs, max_new_tokens: int = 100, device="cuda:0", with_mtp: bool = False,
                  tokenizer=None, eos_id: int = -1, sampling_seed: int = 0, max_seq_len: int | None = None):
         self.config, self.max_new_tokens, self.with_mtp = model_args, max_new_tokens, with_mtp
@@ -34,18 +33,6 @@ class DSAv32Generator:
     def update_sampling_config(self, temperature=0.0, top_p=1.0, top_k=0, use_topp=False) -> None:
         self.decode_layer.update_sampling_config(temperature=temperature, top_p=top_p, top_k=top_k, use_topp=use_topp)
 
-    def _tokens_of(self, prompt, prompt_tokens):
-        if prompt_tokens is not None:
-            return list(prompt_tokens)
-        if self.tokenizer is None:
-            raise ValueError("no tokenizer: pass prompt_tokens=[...]")
-        return self.tokenizer.apply_chat_template([{"role": "user", "content": prompt}], add_generation_prompt=True)
-
-    def _text_of(self, toks: list[int]) -> str:
-        if self.tokenizer is not None:
-            return self.tokenizer.decode(toks, skip_special_tokens=True)
-        return " ".join(str(t) for t in toks)
-
     @torch.inference_mode()
     def generate(self, prompt: str = "", print_log: bool = True, with_mtp: bool | None = None,
                  prompt_tokens: list[int] | None = None) -> tuple[str, list[float], list[int], int]:
@@ -57,33 +44,29 @@ class DSAv32Generator:
         toks = self._tokens_of(prompt, prompt_tokens)
         if active_mtp:
             return self._generate_with_mtp(toks, print_log)
-        return self._generate_without_mtp(toks, print_log)
+        return self._generate_plain(toks, print_log)
 
-    def _generate_without_mtp(self, prompt_tokens: list[int], print_log: bool):
-        """generator.py:187-265."""
-        prompt_len = len(prompt_tokens)
-        total_len = min(self.decode_layer.max_seq_len, self.max_new_tokens + prompt_len)
-        tokens = list(prompt_tokens) + [-1] * (total_len - prompt_len)
-        time_list: list[float] = []
-        for cur in range(1, total_len):
+    # -- the plain loop's steps (generator.py:187-265): the prompt goes through the decode step token by token --
+    def _max_len(self) -> int:
+        return self.decode_layer.max_seq_len
+
+    def _next(self, token: int) -> int:
+        intermediates, *_ = self.decode_layer.forward(token)[0]
+        return int(intermediates[Idx.TOKEN_OUT].view(-1)[0])  # the read synchronises, as the reference's does
+
+    def _prompt(self, tokens: list[int], times: list[float]) -> int:
+        nxt = -1
+        for tok in tokens:
             t0 = time.time()
-            intermediates, *_ = self.decode_layer.forward(tokens[cur - 1])[0]
-            nxt = int(intermediates[Idx.TOKEN_OUT].view(-1)[0])  # the read synchronises, as the reference's does
-            time_list.append(time.time() - t0)
-            if cur >= prompt_len:
-                tokens[cur] = nxt
-                if print_log:
-                    print(self._text_of([nxt]), end=" ", flush=True)
-                if nxt == self.eos_id:
-                    tokens = tokens[: cur + 1]
-                    break
+            nxt = self._next(tok)
+            times.append(time.time() - t0)
+        return nxt
+
+    def vocab_size(self) -> int:
+        return self.config.vocab_size
+
+    def _end_sequence(self) -> None:
         self.decode_layer.reset_sequence()
-        out = [t for t in tokens[prompt_len:] if t != -1]
-        if self.eos_id in out:
-            out = out[: out.index(self.eos_id)]
-        if print_log:
-            print()
-        return self._text_of(out) + "\n", time_list, [], prompt_len
 
     def _generate_with_mtp(self, prompt_tokens: list[int], print_log: bool):
         """generator.py:267-417: chunked prefill of four, then draft / verify / accept steps."""

@@ -7,6 +7,7 @@ from __future__ import annotations
 
 import torch
 
+from ..driver import SequenceDriver
 from . import ops
 from .layer import DecoderLayer, LayerScratch, LayerWeights, precompute_freqs
 from .model_args import ModelArgs
@@ -16,7 +17,9 @@ F32 = torch.float32
 I32 = torch.int32
 
 
-class DsaModel:
+class DsaModel(SequenceDriver):
+    decode_past_last = True  # (the caches then hold every generated token, as the reference's loop leaves them)
+
     def __init__(self, args: ModelArgs, sd: dict[str, torch.Tensor], device="cuda", cache_len: int | None = None,
                  world: int = 1, rank: int = 0, comm: int | None = None, use_graph: bool = True,
                  share_scratch: bool | None = None, temp_vars: list[torch.Tensor] | None = None):
@@ -54,33 +57,14 @@ class DsaModel:
             for li in range(args.n_layers)
         ]
         self.freqs = precompute_freqs(args).to(dev)
-        self.cur_pos = torch.zeros(1, dtype=I32, device=dev)
-        self.token = torch.zeros(1, dtype=torch.int64, device=dev)
-        self.logits = torch.zeros(1, 1, v_l, dtype=F32, device=dev)
-        self.token_out = torch.zeros(1, dtype=torch.int64, device=dev)
+        self._init_sequence(dev, v_l, use_graph)
+        self.full_logits: torch.Tensor | None = None  # world > 1 and sampling: every rank's slice, gathered
         self.temp_vars = temp_vars
         if temp_vars is not None:
             from .temp_var_indices import Idx
 
             self.logits = temp_vars[Idx.LOGITS_OUT].reshape(-1)[:v_l].view(1, 1, v_l)
             self.cur_pos = temp_vars[Idx.CUR_POS].reshape(-1)[:1]
-        self.use_graph = use_graph
-        self._graphs: dict[int, torch.cuda.CUDAGraph] = {}
-        # Host copy of the device-resident position: the kernels write cache row ``cur_pos`` and mask on it,
-        # while the host picks the indexer's scan length from ``pos``; the two must not drift, and a position
-        # past the caches or the rotary table must be refused before anything is launched.
-        self._pos = 0
-        # sampling state (the reference's SAMPLING_CONFIG / TOP_P_SCORES / TOP_N_LOG_PROBS / TOP_N_INDICES
-        # temp vars, temp_var_indices.py:64-73): greedy until set_sampling is called
-        self.sampling_config = torch.tensor([0.0, 1.0, 0.0, 0.0], dtype=F32, device=dev)  # temperature, top_p, top_k, use_top_p
-        self.sampling_seed = 0
-        self.sampling = False
-        self.sample_step = torch.zeros(2, dtype=torch.int64, device=dev)  # advanced by every launch (graph replay safe)
-        self.sampled = torch.zeros(1, dtype=I32, device=dev)
-        self.full_logits: torch.Tensor | None = None  # world > 1 and sampling: every rank's slice, gathered
-        self.token_logprob = torch.zeros(1, dtype=F32, device=dev)
-        self.topn_logprobs = torch.zeros(1, 256, dtype=F32, device=dev)
-        self.topn_indices = torch.zeros(1, 256, dtype=I32, device=dev)
 
     @classmethod
     def from_converted(cls, args: ModelArgs, out_dir, device="cuda", rank: int = 0, **kw) -> "DsaModel":
@@ -90,24 +74,11 @@ class DsaModel:
         packed = convert.load_model(out_dir, device, rank)
         return cls(args, packed, device, world=packed["world"], rank=rank, **kw)
 
-    # -- reference driver controls (end2end.py:551-577) --
-    def reset_sequence(self) -> None:
-        self.cur_pos.zero_()
-        self._pos = 0
-
-    def set_cur_pos(self, pos: int) -> None:
-        if not 0 <= pos < min(self.cache_len, self.freqs.shape[0]):
-            raise ValueError(f"set_cur_pos({pos}): the caches hold {self.cache_len} rows, the rotary table "
-                             f"{self.freqs.shape[0]} positions")
-        self.cur_pos.fill_(pos)
-        self._pos = pos
+    def position_limit(self) -> int:
+        return min(self.cache_len, self.freqs.shape[0])  # rows of the caches, positions of the rotary table
 
     def set_sampling(self, temperature: float = 0.0, top_p: float = 1.0, top_k: int = 0, use_top_p: bool = False,
                      seed: int | None = None) -> None:
-        """Sample the next token instead of taking the arg-max (end2end.py:253-311: temperature, top-p, top-k
-        per request; ``set_sampling_seed``).  Temperature 0 with no seed change returns to greedy decoding.
-        The token's log-probability and the top-256 log-probabilities / ids are left in ``token_logprob``,
-        ``topn_logprobs`` and ``topn_indices`` after every step."""
         if self.world > 1:
             import torch.distributed as dist
 
@@ -116,19 +87,7 @@ class DsaModel:
                                  "torch.distributed: initialise the default process group first")
             if self.full_logits is None:
                 self.full_logits = torch.zeros(self.args.vocab_size, dtype=F32, device=self.device)
-        self.sampling_config.copy_(torch.tensor([temperature, top_p, float(top_k), 1.0 if use_top_p else 0.0]))
-        if seed is not None and seed != self.sampling_seed:
-            self.sampling_seed = seed
-            self._graphs.clear()  # the seed is a launch argument
-        if not self.sampling:
-            self.sampling = True
-            self._graphs.clear()
-
-    def set_sampling_seed(self, seed: int) -> None:
-        """end2end.py:120-134."""
-        if seed != self.sampling_seed:
-            self.sampling_seed = seed
-            self._graphs.clear()
+        super().set_sampling(temperature, top_p, top_k, use_top_p, seed)
 
     def inject_cache(self, layer_caches, start_pos: int = 0, end_pos: int | None = None) -> None:
         """``layer_caches``: one (ki, kv, pe) bf16 triple per layer from an external prefill
@@ -162,13 +121,8 @@ class DsaModel:
         elif self.world > 1:
             # every rank holds vocab / world rows of the head: exchange (value, index) pairs over peer memory
             ops.argmax_exchange(self.logits, self.rank * self.logits.shape[-1], self.token_out, comm=self.comm)
-        elif self.sampling:
-            ops.sample(self.logits.view(1, -1), self.sampling_config, self.sampled, seed=self.sampling_seed,
-                       step=self.sample_step, token_logprob=self.token_logprob, topn_logprobs=self.topn_logprobs,
-                       topn_indices=self.topn_indices)
-            self.token_out.copy_(self.sampled)
         else:
-            self.token_out.copy_(torch.argmax(self.logits.view(-1)))
+            self._choose(self.logits.view(1, -1))
         if self.temp_vars is not None:
             from .temp_var_indices import Idx
 
@@ -176,56 +130,12 @@ class DsaModel:
             self.temp_vars[Idx.TOKEN_ID].view(-1)[:1].copy_(self.token)
         self.cur_pos += 1
 
-    def _bucket(self, pos: int) -> int:
+    def _graph_key(self, pos: int) -> int:
         """Indexer scan length: next multiple of 256 above the position, so graphs are reused."""
         return min(self.cache_len, (pos // 256 + 1) * 256)
 
-    def forward(self, token: int | torch.Tensor, pos: int) -> None:
-        """Run one decode step for ``token`` at position ``pos`` (asynchronous; results in
-        ``self.logits`` / ``self.token_out``)."""
-        if pos != self._pos:
-            raise ValueError(f"forward(pos={pos}): the device position is {self._pos} (use set_cur_pos to move it)")
-        if pos >= self.cache_len or pos >= self.freqs.shape[0]:
-            raise ValueError(f"forward(pos={pos}): past the end of the caches ({self.cache_len} rows) or of the rotary "
-                             f"table ({self.freqs.shape[0]} positions)")
-        if isinstance(token, int):
-            self.token.fill_(token)
-        else:
-            self.token.copy_(token.view(-1)[:1])
-        self._pos = pos + 1
-        n_keys = self._bucket(pos)
-        if not self.use_graph or (self.sampling and self.world > 1):  # the gather is a library collective: not captured
-            self._step_ops(n_keys)
-            return
-        if n_keys not in self._graphs:
-            saved, saved_step = self.cur_pos.clone(), self.sample_step.clone()
-            self._step_ops(n_keys)  # warm-up outside capture (lazy function attributes, allocator)
-            torch.cuda.synchronize()
-            self.cur_pos.copy_(saved)
-            self.sample_step.copy_(saved_step)  # the warm-up drew a number: give it back
-            g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
-                self._step_ops(n_keys)
-            self.cur_pos.copy_(saved)
-            self._graphs[n_keys] = g
-        self._graphs[n_keys].replay()
+    def _sample_op(self):
+        return ops.sample
 
-    @torch.no_grad()
-    def generate(self, prompt: list[int], n_new: int, collect_logits: bool = False):
-        """Token-by-token prefill then greedy decoding (tilert/models/deepseek_v3_2/generator.py:187-265).
-        Returns the generated tokens (and the f32 logits of each generated position)."""
-        self.reset_sequence()
-        pos = 0
-        for tok in prompt:
-            self.forward(tok, pos)
-            pos += 1
-        toks, lgs = [], []
-        for _ in range(n_new):
-            if collect_logits:
-                lgs.append(self.logits.view(-1).clone())
-            nxt = self.token_out.clone()
-            toks.append(nxt)
-            self.forward(nxt, pos)
-            pos += 1
-        toks = [int(t) for t in torch.cat(toks).cpu()]
-        return (toks, lgs) if collect_logits else toks
+    def _may_capture(self) -> bool:
+        return self.use_graph and not (self.sampling and self.world > 1)  # the gather is a library collective: not captured

@@ -169,3 +169,36 @@ def random_packed_model(args: ModelArgs, device, world: int = 1, rank: int = 0, 
                "w_eh": (torch.randn(a.dim, 2 * a.dim, generator=gen, device=dev) * 0.01).to(BF16), "norm": ones.clone()}
     return {"layers": [random_packed_layer(a, li, dev, world, rank, seed) for li in range(a.n_layers)], "world": world,
             "embed": embed, "final_norm": ones, "head": head, "mtp": mtp}
+
+
+def random_ralasun_state_dict(args, device="cpu", seed: int = 0) -> dict[str, torch.Tensor]:
+    """A random-init Ralasun model under its checkpoint names: projections of variance 1 / fan-in, norm weights
+    around their neutral value, router biases, mixing factors between 0 and 1 -- nothing left at a value that would
+    hide a missing term."""
+    dev = torch.device(device)
+    gen = torch.Generator(device=dev).manual_seed(seed)
+
+    def rnd(*shape, std=1.0, mean=0.0):
+        return (torch.randn(*shape, generator=gen, dtype=torch.float32, device=dev) * std + mean).to(BF16)
+
+    def lin(n, k):
+        return rnd(n, k, std=k ** -0.5)
+
+    d = args.dim
+    sd = {"embed": rnd(args.vocab_size, d), "embed.norm": rnd(d, std=0.2), "final.norm": rnd(d, std=0.2), "head": lin(args.vocab_size, d)}
+    for i, layer in enumerate(args.layers):
+        m, f = layer.mixer, layer.mlp
+        nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
+        p = f"l{i}"
+        sd |= {f"{p}.norm1": rnd(d, std=0.2), f"{p}.mix.q": lin(nq, d), f"{p}.mix.k": lin(nk, d), f"{p}.mix.v": lin(nv, d),
+               f"{p}.mix.q.norm": rnd(nq, std=0.2, mean=1.3), f"{p}.mix.k.norm": rnd(nk, std=0.2, mean=1.3),
+               f"{p}.mix.vmix": (torch.rand((), generator=gen, device=dev) * 0.6 + 0.2).to(BF16), f"{p}.mix.o": lin(d, m.heads * m.vdim)}
+        if f is None:
+            continue
+        sd |= {f"{p}.norm2": rnd(d, std=0.2), f"{p}.mlp.router": lin(f.experts, d), f"{p}.mlp.router.b": rnd(f.experts, std=0.5)}
+        for e in range(f.experts):
+            sd |= {f"{p}.mlp.e{e}.gate": lin(f.ff, d), f"{p}.mlp.e{e}.up": lin(f.ff, d), f"{p}.mlp.e{e}.down": lin(d, f.ff)}
+        if f.shared_ff:
+            sd |= {f"{p}.mlp.shared.gate": lin(f.shared_ff, d), f"{p}.mlp.shared.up": lin(f.shared_ff, d),
+                   f"{p}.mlp.shared.down": lin(d, f.shared_ff)}
+    return sd

@@ -1,0 +1,89 @@
+"""Replays a trace of given token ids through a model, step by step, and writes the logits that are asked for.
+
+    bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR [--max-tokens N]
+
+Standard input holds one JSON object per line,
+
+    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["a"]}
+
+and every step's wanted logits go to OUT/<step>.f32 (little-endian f32, [wanted, vocab]); "done <step>" is printed when a
+step has been run.  Nothing is sampled.  The model runs one sequence at a time: a request's tokens continue where its
+last step ended, and a new request may begin once the one before it has been ended.  Exit code 3: the model does not
+run in the asked-for type.
+"""
+
+from __future__ import annotations
+
+import argparse
+import json
+import sys
+from pathlib import Path
+
+
+class TraceRunner:
+    """Steps of a trace on one ``SequenceDriver``."""
+
+    def __init__(self, model):
+        self.model = model
+        self.active = None  # id of the request the model's sequence belongs to
+
+    def step(self, entries: list[dict], end: list):
+        """Run a step's entries; returns the wanted logits [wanted, vocab] or None."""
+        import torch
+
+        outs = []
+        for e in entries:
+            if self.active is None:
+                self.model.reset_sequence()
+                self.active = e["id"]
+            elif self.active != e["id"]:
+                raise ValueError(f"request {e['id']!r} while {self.active!r} is live: the model holds one sequence")
+            tokens, want = [int(t) for t in e["tokens"]], [int(w) for w in e.get("want", [])]
+            if tokens:
+                outs.append(self.model.prefill(tokens, want))
+        for rid in end:
+            if rid != self.active:
+                raise ValueError(f"request {rid!r} is not live")
+            self.active = None
+            self.model.reset_sequence()
+        outs = [o for o in outs if o.shape[0]]
+        return torch.cat(outs) if outs else None
+
+
+def main(argv=None) -> int:
+    ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
+    ap.add_argument("--model", required=True, help="directory with config.json and model.safetensors")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
+    ap.add_argument("--out", required=True, help="directory for the logits")
+    ap.add_argument("--max-tokens", type=int, default=None, help="most tokens that live requests hold at any time")
+    a = ap.parse_args(argv)
+
+    from tilert_b200.models.registry import family_of_dir
+
+    family = family_of_dir(a.model)
+    if a.dtype not in family.dtypes:
+        print(f"{family.name} runs in {', '.join(family.dtypes)}, not in {a.dtype}", file=sys.stderr)
+        return 3
+    from tilert_b200 import build
+
+    build.build(model_type=family.name)  # a fresh checkout has no libraries yet
+    import tilert_b200 as tb
+
+    model = family.load(a.model, "cuda:0", a.dtype, a.max_tokens)
+    runner, out = TraceRunner(model), Path(a.out)
+    for line in sys.stdin:
+        if not line.strip():
+            continue
+        s = json.loads(line)
+        logits = runner.step(s["entries"], s.get("end", []))
+        if logits is not None:
+            (out / f"{s['step']}.f32").write_bytes(logits.float().cpu().contiguous().numpy().astype("<f4").tobytes())
+        status = tb.device_status(0, model.backend)
+        if status != 0:
+            raise RuntimeError(f"a kernel gave up with status {status}")
+        print(f"done {s['step']}", flush=True)
+    return 0
+
+
+if __name__ == "__main__":
+    sys.exit(main())
