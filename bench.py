@@ -724,6 +724,267 @@ def run_c3(args) -> None:
         sys.exit(1)
 
 
+RALASUN_SIZES = {
+    # name: width, query heads, kv heads, experts, top, expert ff, shared ff, window (head sizes 128 / 128), closest model's q_lora
+    "w2048": (2048, 16, 4, 64, 6, 1408, 2816, 1024, 768),
+    "w4096": (4096, 32, 8, 64, 8, 1536, 1536, 2048, 1536),
+    "w7168": (7168, 64, 8, 48, 8, 2048, 2048, 4096, 1536),
+}
+
+
+def _graph_us(fn, reps: int) -> float:
+    """Microseconds per call of ``fn`` replayed from a CUDA graph (median of ``reps`` replays)."""
+    for _ in range(2):
+        fn()
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        fn()
+    for _ in range(3):
+        g.replay()
+    ts = []
+    for _ in range(reps):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        g.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        ts.append(e0.elapsed_time(e1) * 1e3)
+    return sorted(ts)[len(ts) // 2]
+
+
+def _ralasun_arm(size, n_layers: int, portion: int, reps: int) -> dict:
+    """Decode and prefill of a stack of equal Ralasun layers, and each of its kernels over the stack's weights."""
+    from tilert_b200 import gqa_ops as go
+    from tilert_b200 import synthetic
+    from tilert_b200.models.ralasun.layer import Pending, Stream
+    from tilert_b200.models.ralasun.model import RalasunModel
+    from tilert_b200.models.ralasun.model_args import GATE_ALPHA, MixerArgs, MlpArgs, uniform_args
+
+    width, heads, kv, experts, top, ff, sff, window, _ = size
+    mix = MixerArgs(heads, kv, 128, 128, window, 128 ** -0.5, True)
+    args = uniform_args(n_layers, width, 32768, mix, MlpArgs(experts, top, ff, 7.0, sff, 7.0), max_seq_len=3 * max(window, portion))
+    sd = synthetic.random_ralasun_state_dict(args, "cuda", seed=0)
+    model = RalasunModel(args, sd, "cuda", portion=portion)
+    del sd
+    torch.cuda.empty_cache()
+    toks = torch.randint(0, args.vocab_size, (portion,), generator=torch.Generator().manual_seed(1)).tolist()
+    start = max(window, portion) // portion * portion  # a full window of cached keys before anything is timed
+
+    # ---- prefill of one portion behind a full window ----
+    ts = []
+    for i in range(2 + max(reps // 4, 5)):
+        model.reset_sequence()
+        while model._pos < start:
+            model.prefill(toks, [])
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        model.prefill(toks, [])
+        e1.record()
+        torch.cuda.synchronize()
+        ts.append(e0.elapsed_time(e1))
+    prefill_ms = sorted(ts[2:])[len(ts[2:]) // 2]
+    flops = portion * n_layers * 2 * (width * (heads * 128 + 2 * kv * 128) + heads * 128 * width + 3 * width * (top * ff + sff) + width * experts) \
+        + portion * n_layers * 4 * heads * 128 * window + 2 * width * args.vocab_size
+
+    # ---- decode ----
+    tok = torch.tensor([1], dtype=torch.int64, device="cuda")
+    for _ in range(5):
+        model.forward(tok, model._pos)
+    ts = []
+    for _ in range(reps):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        model.forward(tok, model._pos)
+        e1.record()
+        torch.cuda.synchronize()
+        ts.append(e0.elapsed_time(e1) * 1e3)
+    step_us = sorted(ts)[len(ts) // 2]
+    kv_bytes = 2 * kv * 128 * window * 2
+    step_bytes = model.weight_bytes() + n_layers * kv_bytes
+
+    # ---- the kernels one by one, each over all layers' weights in one graph ----
+    peak, _src = _peak_gbs()
+    kernels = {}
+
+    def add(name, fn, nbytes=None, nflops=None):
+        us = _graph_us(lambda: [fn(layer) for layer in model.layers], reps) / n_layers
+        k = {"us": round(us, 2)}
+        if nbytes:
+            k |= {"bytes": nbytes, "frac_hbm": round(nbytes / us / 1e3 / peak, 3)}
+        if nflops:
+            k |= {"tflops": round(nflops / us / 1e6, 1), "frac_tensor": round(nflops / us / 1e6 / peak_tflops(), 3)}
+        kernels[name] = k
+
+    a, sc, f, eps = args, model.scratch, args.layers[0].mlp, args.eps
+    nq, nqkv = heads * 128, heads * 128 + 2 * kv * 128
+    st = Stream(sc, width)
+    vq, vy, va = sc.get("vec_qkv", nqkv), sc.get("vec_y", width), sc.get("vec_att", nq)
+    vl, vh = sc.get("vec_router", go.pad(experts)), sc.get("vec_hidden", go.pad(sff) + top * go.pad(ff))
+    vi, vw = sc.get("vec_ids", top, dtype=torch.int32), sc.get("vec_w", top)
+
+    def qkv1(layer):
+        st.pending = Pending(vy, layer.w.norm2)
+        st.dense(layer.w.qkv, vq, nqkv, width, eps)
+
+    def attn1(layer):
+        n = min(layer.max_splits, (window + 63) // 64)
+        go.vec_attn(vq, layer.w.q_gain, layer.w.k_gain, eps, 0, None, None, mix, layer.cache, model.cur_pos, n,
+                    sc.get("vec_part", heads * n * 130), sc.get("vec_counter", layer.head_blocks, dtype=torch.int32), va)
+
+    def router1(layer):
+        st.pending = Pending(vy, layer.w.norm1)
+        st.dense(layer.w.router, vl, experts, width, eps, bias=layer.w.router_bias)
+
+    add("decode qkv (+ norm, residual)", qkv1, nqkv * width * 2)
+    add("decode attention (+ q/k norm, cache write)", attn1, kv_bytes)
+    add("decode output product", lambda l: go.vec_dense(va, l.w.o, vy, width, nq), nq * width * 2)
+    add("decode router (+ norm, residual)", router1, experts * width * 2)
+    add("decode gate/up (+ routing)", lambda l: go.vec_gate_up(st.x, width, vl, top, l.w.gate_up, l.w.shared_gate_up, ff, sff, 7.0, 7.0, GATE_ALPHA,
+                                                               vh, vi, vw), 4 * width * (top * ff + sff))
+    add("decode down", lambda l: go.vec_down(vh, vi, vw, top, l.w.down, l.w.shared_down, ff, sff, width, vy), 2 * width * (top * ff + sff))
+
+    p, bf = portion, torch.bfloat16
+    x, xh = sc.get("x", p, width), sc.get("xh", p, width, dtype=bf)
+    qkv, q, att = sc.get("qkv", p, nqkv), sc.get("q", p, heads, 128, dtype=bf), sc.get("att", p, nq, dtype=bf)
+    y, logits = sc.get("y", p, width), sc.get("router", p, go.pad(experts))
+    ids, rank, slot = (sc.get(n, p, top, dtype=torch.int32) for n in ("ids", "rank", "slot_row"))
+    sw, counts = sc.get("slot_w", p, top), sc.get("counts", experts, dtype=torch.int32)
+    xs, hid, ye = sc.get("xs", p * top, width, dtype=bf), sc.get("hid", p * top, ff, dtype=bf), sc.get("ye", p * top, width, dtype=bf)
+    hsh, ysh = sc.get("hsh", p, sff, dtype=bf), sc.get("ysh", p, width, dtype=bf)
+    model.set_cur_pos(start)
+    x.normal_()
+    xh.copy_(x)
+    add("prefill qkv", lambda l: go.gemm(xh, l.w.qkv, qkv, p, nqkv, width), None, 2 * p * nqkv * width)
+    add("prefill q/k norm, cache write", lambda l: go.qkv_rows(qkv, l.w.q_gain, l.w.k_gain, eps, 0, None, None, p, mix, l.cache, model.cur_pos, q),
+        p * nqkv * 6)
+    add("prefill attention", lambda l: go.attn_rows(q, mix, l.cache, model.cur_pos, p, att), None, 4 * p * heads * 128 * window)
+    add("prefill output product", lambda l: go.gemm(att, l.w.o, y, p, width, nq), None, 2 * p * nq * width)
+    add("prefill router", lambda l: go.gemm(xh, l.w.router, logits, p, experts, width, bias=l.w.router_bias), p * width * 2 + experts * width * 2)
+    add("prefill routing", lambda l: go.route_rows(logits, p, experts, top, ids, sw, rank, counts))
+    add("prefill gather", lambda l: go.gather_rows(xh, p, width, experts, top, ids, rank, counts, xs, slot), p * width * 2 * (1 + top))
+    add("prefill experts gate/up", lambda l: go.gemm(xs, l.w.gate_up, hid, p * top, ff, width, gated=(7.0, GATE_ALPHA), n_groups=experts, counts=counts),
+        None, 4 * p * top * ff * width)
+    add("prefill experts down", lambda l: go.gemm(hid, l.w.down, ye, p * top, width, ff, n_groups=experts, counts=counts), None, 2 * p * top * ff * width)
+    add("prefill shared gate/up", lambda l: go.gemm(xh, l.w.shared_gate_up, hsh, p, sff, width, gated=(7.0, GATE_ALPHA)), None, 4 * p * sff * width)
+    add("prefill shared down", lambda l: go.gemm(hsh, l.w.shared_down, ysh, p, width, sff), None, 2 * p * sff * width)
+    add("prefill combine, norm, residual", lambda l: go.residual_norm(x, xh, l.w.norm2, eps, width, p, experts=ye, slot_row=slot, slot_w=sw, shared=ysh),
+        p * width * (2 * (top + 1) + 10))
+    out = torch.empty(p, nqkv, dtype=bf, device="cuda")
+    us = _graph_us(lambda: [torch.matmul(xh, l.w.qkv.T, out=out) for l in model.layers], reps) / n_layers
+    kernels["(cuBLAS, the qkv product's shape)"] = {"us": round(us, 2), "tflops": round(2 * p * nqkv * width / us / 1e6, 1)}
+    import tilert_b200
+
+    return {"decode_us_per_step": step_us, "decode_tokens_per_s": 1e6 / step_us, "decode_bytes": step_bytes,
+            "decode_frac_hbm": step_bytes / step_us / 1e3 / peak, "decode_us_per_layer": step_us / n_layers,
+            "prefill_ms_per_portion": prefill_ms, "prefill_tokens_per_s": portion / prefill_ms * 1e3,
+            "prefill_tflops": flops / prefill_ms / 1e9, "prefill_frac_tensor": flops / prefill_ms / 1e9 / peak_tflops(),
+            "kernels": kernels, "device_status": tilert_b200.device_status(0, "ralasun")}
+
+
+def peak_tflops() -> float:
+    pk = ROOT / "MEASURED_PEAKS.json"
+    return float(json.loads(pk.read_text())["bf16_tflops"]) if pk.exists() else 1590.0
+
+
+def _closest_arm(size, n_layers: int, reps: int) -> dict:
+    """The DeepSeek-V3.2-style layers of this framework at the same width, heads, experts and expert sizes (its own
+    attention), decoding; its prompts go four rows per step."""
+    from dataclasses import replace
+
+    import tilert_b200
+    from tilert_b200 import synthetic
+    from tilert_b200.models.deepseek_v3_2 import layer as L
+    from tilert_b200.models.deepseek_v3_2 import ops
+    from tilert_b200.models.deepseek_v3_2.model_args import ModelArgs
+
+    width, heads, _, experts, top, ff, _, window, q_lora = size
+    ctx = max(window, 2048) + 256
+    a = replace(ModelArgs(), dim=width, n_heads=heads, n_layers=n_layers, n_dense_layers=0, n_routed_experts=experts, n_activated_experts=top,
+                moe_inter_dim=ff, n_expert_groups=1, n_limited_groups=1, q_lora_rank=q_lora, vocab_size=32768, max_seq_len=ctx, index_n_heads=16)
+    dev = torch.device("cuda", 0)
+    peak, _ = _peak_gbs()
+    ws = [synthetic.random_packed_layer(a, li, dev, seed=0) for li in range(n_layers)]
+    out = {}
+    for rows in (1, 4):
+        scratch = L.LayerScratch(a, dev, ctx, rows)
+        layers = [L.DecoderLayer(a, w, dev, ctx, rows, scratch=scratch, out_slot=i) for i, w in enumerate(ws)]
+        for layer in layers:
+            for t in (layer.kv_cache, layer.pe_cache, layer.ki_cache):
+                t.normal_()
+        cur = torch.tensor([ctx - rows], dtype=torch.int32, device=dev)
+        freqs = L.precompute_freqs(a)[ctx - rows: ctx].contiguous().to(dev)
+        x = torch.randn(1, rows, width, device=dev).to(torch.bfloat16)
+
+        def stack():
+            h = x
+            for layer in layers:
+                h = layer.forward(h, cur, freqs, ctx)
+        us = _graph_us(stack, reps)
+        nbytes = sum(w.weight_bytes(a) for w in ws) + n_layers * (a.index_topk * 576 * 2 + ctx * 256)
+        if rows == 1:
+            out |= {"decode_us_per_layer": us / n_layers, "decode_tokens_per_s": 1e6 / us, "decode_bytes": nbytes,
+                    "decode_frac_hbm": nbytes / us / 1e3 / peak}
+            kernels = {}
+
+            def add(name, fn, nb):
+                t = _graph_us(lambda: [fn(layer) for layer in layers], reps) / n_layers
+                kernels[name] = {"us": round(t, 2), "bytes": int(nb), "frac_hbm": round(nb / t / 1e3 / peak, 3)}
+            w0 = ws[0]
+            per = (w0.w_gu[0].numel(), w0.w_down[0].numel())
+            add("decode q_a / kv_a (+ norm)", lambda l: ops.rmsnorm_projx_wqkva(x, l.w.in_norm, l.w.w_qkva, cur, l.q_a, l.kv, l.pe_cache, l.ki, eps=a.eps),
+                w0.w_qkva.numel())
+            add("decode q_b (+ norm)", lambda l: ops.rmsnorm_proj_q(l.q_a, l.w.q_norm, l.w.w_qb, l.q_nope, l.q_pe, l.iq, eps=a.eps), w0.w_qb.numel())
+            add("decode sparse attention (+ value product)", lambda l: ops.flash_sparse_mla(
+                l.q_lat, l.q_pe, l.kv_cache, l.pe_cache, l.sel, cur, l.o_lat, softmax_scale=l.scale, split_size=l.mla_split, out_acc=l.o_acc,
+                lse=l.lse, lse_acc=l.lse_acc, w_v=l.w.w_v, o_out=l.o), a.index_topk * 576 * 2 + w0.w_v.numel())
+            add("decode output product (+ residual)", lambda l: ops.unproj_o_allreduce(l.o, l.w.w_o, None, x, 0, l.h), w0.w_o.numel())
+            add("decode router (+ norm)", lambda l: ops.rmsnorm_expert_proj(l.h, l.w.post_norm, l.w.router, l.scores, l.h_norm, eps=a.eps),
+                w0.router.numel() * 2)
+            add("decode gate/up (+ routing)", lambda l: ops.expert_select_up_gate_silu(
+                l.h_norm, l.scores, l.w.router_bias, l.w.w_gu, l.ffn_hidden, l.probs, l.eidx, dim=a.dim, n_groups=1, n_limited_groups=1,
+                route_scale=a.route_scale, slot_ids=l.slot_ids, slot_w=l.slot_w), (top + 1) * per[0])
+            add("decode down (+ residual)", lambda l: ops.expert_down_allreduce(l.ffn_hidden, l.w.w_down, None, l.eidx, l.probs, l.h, 0, l.out,
+                                                                                slot_ids=l.slot_ids, slot_w=l.slot_w), (top + 1) * per[1])
+            out["kernels"] = kernels
+        else:
+            out |= {"prefill_tokens_per_s": rows * 1e6 / us, "prefill_rows_per_step": rows, "prefill_us_per_step": us}
+        del layers, scratch
+    out["device_status"] = tilert_b200.device_status(0)
+    return out
+
+
+def run_ralasun(args) -> None:
+    """Layers of the Ralasun design at sizes that resemble a real model's, beside the framework's closest model at
+    equal size: decode and prefill throughput, and every kernel's time and fraction of its roofline.  The weights of a
+    timed pass exceed the L2 several times over.  One JSON line per size; random weights."""
+    import tilert_b200
+
+    for be in ("deepseek_v3_2", "ralasun"):
+        tilert_b200.load_backend(be)
+        tilert_b200.tilert_init(0, be)
+    names = args.sizes.split(",") if args.sizes else list(RALASUN_SIZES)
+    n_layers, portion, reps = 6, 2048, max(args.steps, 10)
+    for name in names:
+        size = RALASUN_SIZES[name]
+        sampler = ClockSampler(0)
+        sampler.start()
+        ours = _ralasun_arm(size, n_layers, portion, reps)
+        clocks = sampler.stop()
+        torch.cuda.empty_cache()
+        closest = _closest_arm(size, n_layers, reps)
+        torch.cuda.empty_cache()
+        print(json.dumps({
+            "metric": "ralasun_decode_tokens_per_s", "value": ours["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": reps,
+            "ms_per_step": ours["decode_us_per_step"] * 1e-3, "higher_is_better": True, "dtype": "bf16 weights, f32 accumulate", "data": "synthetic",
+            "config": {"size": name, "layers": n_layers, "width": size[0], "heads": size[1], "kv_heads": size[2], "experts": size[3], "top": size[4],
+                       "expert_ff": size[5], "shared_ff": size[6], "window": size[7], "portion": portion, "vocab": 32768,
+                       "l2": "one pass reads every layer's own weights: several times the L2", "peak_hbm_gbs": _peak_gbs()[0],
+                       "peak_source": _peak_gbs()[1], "peak_bf16_tflops": peak_tflops()},
+            "ralasun": ours, "closest": {"model": "deepseek_v3_2 layers, FP8 weights, same width / heads / experts", **closest}, "clocks": clocks}), flush=True)
+
+
 def run_profile_gemv(args) -> None:
     """One weight-streaming product alone: N = 7168 rows, K = 32768 (235 MB of FP8 weights, larger
     than L2), a few launches.  Small device footprint, meant to be captured by a profiler."""
@@ -819,15 +1080,16 @@ def main() -> None:
                     help="short run for a profiler: no clock-sampling loop, no CPU baseline")
     ap.add_argument("--trace-step", action="store_true",
                     help="print the per-launch phase stamps of the streaming products of one step")
-    ap.add_argument("--config", default="c1", choices=["c1", "c2", "c3"],
+    ap.add_argument("--config", default="c1", choices=["c1", "c2", "c3", "ralasun"],
                     help="c1: the headline layer step; c2: whole-model decode (time per output token); c3: long-context "
-                         "indexer + sparse attention stress")
+                         "indexer + sparse attention stress; ralasun: that design's layers beside the closest model's")
     ap.add_argument("--ctx", default=None, help="c2: context length(s), comma separated (default 1024); c3: cached keys "
                                                 "(default 131072)")
     ap.add_argument("--chain", default="default", choices=["default", "on", "off", "both"],
                     help="c2: run the layers' products as chained launches, as single launches, or time both")
     ap.add_argument("--with-mtp", action="store_true", help="c2: speculative decoding steps with the prediction layer")
     ap.add_argument("--layers", type=int, default=61, help="c2: decoder layers (61 = the real model; needs 8 GPUs)")
+    ap.add_argument("--sizes", default=None, help="ralasun: comma separated sizes (default: all)")
     ap.add_argument("--gemv-k", type=int, default=32768)
     ap.add_argument("--gemv-packed", action="store_true", help="profile-gemv: activations packed beforehand")
     ap.add_argument("--profile-gemv", action="store_true",
@@ -841,6 +1103,8 @@ def main() -> None:
     elif args.config == "c3" and args.impl == "ours":
         args.ctx = int(args.ctx or 131072)
         run_c3(args)
+    elif args.config == "ralasun" and args.impl == "ours":
+        run_ralasun(args)
     elif args.profile_gemv:
         run_profile_gemv(args)
     elif args.impl == "reference":

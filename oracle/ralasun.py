@@ -71,6 +71,12 @@ def route(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, top: int) -> tup
     return ids, torch.softmax(z[ids], dim=0)
 
 
+def route_margin(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, top: int) -> float:
+    """Distance between the last chosen logit and the first that is not (how close a call the routing is)."""
+    z = torch.sort(w @ x + bias, descending=True).values
+    return float(z[top - 1] - z[top]) if top < z.numel() else float("inf")
+
+
 def mixture(x: torch.Tensor, w: dict, p: str, mlp: dict) -> torch.Tensor:
     """Weighted sum of the chosen experts, plus the shared one; token by token."""
     out = torch.zeros_like(x)
@@ -101,8 +107,11 @@ def mixer(x: torch.Tensor, w: dict, p: str, mix: dict, eps: float, first: list) 
     return o.reshape(t, h * dv) @ w[f"{p}.o"].T
 
 
-def forward(cfg: dict, weights: dict, tokens: list[int], dtype=torch.float64, layers_out: list | None = None) -> torch.Tensor:
-    """Logits [T, vocab] of one whole sequence; ``layers_out`` receives the residual stream after every layer."""
+def forward(cfg: dict, weights: dict, tokens: list[int], dtype=torch.float64, layers_out: list | None = None,
+            margins: list | None = None) -> torch.Tensor:
+    """Logits [T, vocab] of one whole sequence; ``layers_out`` receives the residual stream after every layer,
+    ``margins`` every token's smallest routing margin over the layers."""
+    closest = torch.full((len(tokens),), float("inf"))
     w = {k: t.to(dtype) for k, t in weights.items()}
     eps = cfg["norm"]["eps"]
     x = norm_around_one(w["embed"][torch.tensor(tokens)], w["embed.norm"], eps)
@@ -110,7 +119,13 @@ def forward(cfg: dict, weights: dict, tokens: list[int], dtype=torch.float64, la
     for i, layer in enumerate(cfg["layers"]):
         x = x + norm_around_one(mixer(x, w, f"l{i}.mix", layer["mixer"], eps, first), w[f"l{i}.norm1"], eps)
         if layer.get("mlp") is not None:
+            if margins is not None:
+                m, top = f"l{i}.mlp", layer["mlp"]["router"]["top"]
+                here = [route_margin(r, w[f"{m}.router"], w[f"{m}.router.b"], top) for r in x]
+                closest = torch.minimum(closest, torch.tensor(here))
             x = x + norm_around_one(mixture(x, w, f"l{i}.mlp", layer["mlp"]), w[f"l{i}.norm2"], eps)
         if layers_out is not None:
             layers_out.append(x.clone())
+    if margins is not None:
+        margins.extend(closest.tolist())
     return norm_around_one(x, w["final.norm"], eps) @ w["head"].T

@@ -4,6 +4,7 @@
 
 #include <cuda.h>
 
+#include <cmath>
 #include <mutex>
 
 #include "host_util.h"
@@ -207,14 +208,16 @@ extern "C" int tilert_gqa_gemm_op(TgContext* ctx, const void* x, long long ldx, 
   }
   const long long w_rows = static_cast<long long>(n_groups > 0 ? n_groups : 1) * per * n;
   const int ft = (n + 127) / 128;
-  // the widest token tile that still gives every SM a tile (one weight), or that an average group fills
-  auto fits = [&](int bn) {
-    if (n_groups > 0) return rows / n_groups >= bn * 3 / 4;
-    return static_cast<long long>(ft) * ((rows + bn - 1) / bn) >= ctx->num_sms * 3 / 4;
+  // Token tile: waves of tiles over the SMs times the relative cost of a tile (narrow tiles reuse a weight tile less).
+  // Groups are taken as equally long, each ending in a half-filled tile.
+  auto cost = [&](int bn, double tile) {
+    const double tiles = n_groups > 0 ? ft * (static_cast<double>(rows) / bn + 0.5 * n_groups) : static_cast<double>(ft) * ((rows + bn - 1) / bn);
+    return std::ceil(tiles / ctx->num_sms) * tile;
   };
-  if (gated) return fits(128) ? launch_tc<128, true>(ctx, p, w_rows, stream) : launch_tc<64, true>(ctx, p, w_rows, stream);
-  if (fits(256)) return launch_tc<256, false>(ctx, p, w_rows, stream);
-  if (fits(128)) return launch_tc<128, false>(ctx, p, w_rows, stream);
+  if (gated) return cost(128, 1.0) <= cost(64, 0.6) ? launch_tc<128, true>(ctx, p, w_rows, stream) : launch_tc<64, true>(ctx, p, w_rows, stream);
+  const double c256 = cost(256, 1.0), c128 = cost(128, 0.56), c64 = cost(64, 0.34);
+  if (c256 <= c128 && c256 <= c64) return launch_tc<256, false>(ctx, p, w_rows, stream);
+  if (c128 <= c64) return launch_tc<128, false>(ctx, p, w_rows, stream);
   return launch_tc<64, false>(ctx, p, w_rows, stream);
 }
 
@@ -340,7 +343,7 @@ extern "C" int tilert_gqa_vec_attn_op(TgContext* ctx, const float* qkv, const fl
   const int rc = check_qkv(a.s);
   if (rc != TB_OK) return rc;
   TB_REQUIRE(ctx != nullptr && qkv != nullptr && q_gain != nullptr && k_gain != nullptr && pos != nullptr && k_cache != nullptr &&
-             v_cache != nullptr && out != nullptr && n_splits >= 1 && (n_splits == 1 || (part != nullptr && counter != nullptr)));
+             v_cache != nullptr && out != nullptr && n_splits >= 1 && n_splits <= 1024 && (n_splits == 1 || (part != nullptr && counter != nullptr)));
   TB_REQUIRE(v_mode == VMIX_NONE || v_first != nullptr);
   TB_REQUIRE(v_mode != VMIX_BLEND || lambda != nullptr);
   a.p = {qkv, 0, q_gain, k_gain, eps, v_mode, lambda, v_first};

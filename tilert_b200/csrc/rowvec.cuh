@@ -4,10 +4,11 @@
 //   gate/up   routing, then hidden = clamped_gate(W_gate x, W_up x) of the shared and the selected experts
 //   down      out[d] = sum over slots of w_slot W_down[slot][d, :] . hidden[slot]
 //
-// One CTA of 16 warps per SM.  A CTA owns a contiguous range of weight rows; its warps split K (piece c of eight
-// elements belongs to thread c mod 512), four rows per step with the next two steps' rows already requested, so
-// that 8-12 sixteen-byte loads per thread are in flight.  Four row sums are reduced across a warp together
-// (transposing: six shuffles instead of twenty) and the 16 per-warp sums meet in shared memory at the end.
+// One CTA of 16 warps per SM.  A CTA owns a contiguous range of weight rows.  A team of warps -- all 16, or fewer when
+// K is short -- works on four rows at a time: its threads split K (piece c of eight elements belongs to thread c mod
+// team size) and have the next two steps' rows already requested, so that 8-12 sixteen-byte loads per thread are in
+// flight.  Four row sums are reduced across a warp together (transposing: six shuffles instead of twenty) and the
+// per-warp sums of a team meet in shared memory at the end.
 //
 // The vector is staged once per CTA.  Staging can apply what lies between two sublayers -- x + rms(y) gain, written
 // back by CTA 0, and a further norm on top -- so that the norms and the residual of a decode step need no launches of
@@ -115,48 +116,65 @@ __device__ __forceinline__ uint4 ld_stream(const __nv_bfloat16* p) {
   return v;
 }
 
-// Cursor over the (row group, piece) steps of a CTA.
+// How the CTA's threads share rows of `chunks` pieces: teams of a power of two of warps, the smallest that
+// covers a row in one go (or all of them).
+struct RvTeam {
+  int chunks, warps, threads, n_teams, team, tid, warp, nc;
+  __device__ __forceinline__ explicit RvTeam(int chunks_) : chunks(chunks_) {
+    warps = kRvWarps;
+    while (warps > 1 && chunks <= warps * 16) warps >>= 1;
+    threads = warps * 32;
+    n_teams = kRvWarps / warps;
+    team = threadIdx.x / threads;
+    tid = threadIdx.x - team * threads;
+    warp = tid >> 5;
+    nc = (chunks + threads - 1) / threads;
+  }
+};
+
+// Cursor over the (row group, piece) steps of a team.
 struct RvCursor {
-  int group = 0, ci = 0;
-  __device__ __forceinline__ void next(int nc) {
-    if (++ci == nc) {
+  int group, ci = 0;
+  __device__ __forceinline__ explicit RvCursor(const RvTeam& t) : group(t.team) {}
+  __device__ __forceinline__ void next(const RvTeam& t) {
+    if (++ci == t.nc) {
       ci = 0;
-      ++group;
+      group += t.n_teams;
     }
   }
 };
 
 template <class Src>
-__device__ __forceinline__ void rv_load(const Src& src, const RvCursor& c, int rows, int chunks, uint4 (&w)[kRvRows]) {
-  const int piece = c.ci * kRvThreads + threadIdx.x;
+__device__ __forceinline__ void rv_load(const Src& src, const RvTeam& t, const RvCursor& c, int rows, uint4 (&w)[kRvRows]) {
+  const int piece = c.ci * t.threads + t.tid;
 #pragma unroll
   for (int r = 0; r < kRvRows; ++r) {
     const int row = c.group * kRvRows + r;
-    w[r] = (row < rows && piece < chunks) ? src.load(row, piece) : make_uint4(0u, 0u, 0u, 0u);
+    w[r] = (row < rows && piece < t.chunks) ? src.load(row, piece) : make_uint4(0u, 0u, 0u, 0u);
   }
 }
 
-// Sums of `rows` weight rows (Src::load(row, piece)) against the staged vector into part[row][warp].
+// Sums of `rows` weight rows (Src::load(row, piece)) against the staged vector into part[row][warp of the team].
 // `ahead` holds the first 1 + kRvAhead steps' weights when `loaded` is set.
 template <class Src>
-__device__ __forceinline__ void rv_rows(const Src& src, int rows, int chunks, const RvVec& v, float* part,
+__device__ __forceinline__ void rv_rows(const Src& src, const RvTeam& t, int rows, const RvVec& v, float* part,
                                         uint4 (&ahead)[kRvAhead + 1][kRvRows], bool loaded) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int nc = (chunks + kRvThreads - 1) / kRvThreads;
-  const int steps = (rows + kRvRows - 1) / kRvRows * nc;
-  RvCursor cur, pre;
+  const int lane = threadIdx.x & 31;
+  const int groups = (rows + kRvRows - 1) / kRvRows;
+  const int steps = (groups - t.team + t.n_teams - 1) / t.n_teams * t.nc;  // of this team
+  RvCursor cur(t), pre(t);
 #pragma unroll
   for (int d = 0; d <= kRvAhead; ++d) {
-    if (!loaded) rv_load(src, pre, rows, chunks, ahead[d]);
-    pre.next(nc);
+    if (!loaded) rv_load(src, t, pre, rows, ahead[d]);
+    pre.next(t);
   }
   float acc[kRvRows];
 #pragma unroll
   for (int r = 0; r < kRvRows; ++r) acc[r] = 0.f;
 #pragma unroll 3
   for (int s = 0; s < steps; ++s) {
-    const int piece = cur.ci * kRvThreads + threadIdx.x;
-    if (piece < chunks) {
+    const int piece = cur.ci * t.threads + t.tid;
+    if (piece < t.chunks) {
       const float4 a = reinterpret_cast<const float4*>(v.lo)[piece], b = reinterpret_cast<const float4*>(v.hi)[piece];
 #pragma unroll
       for (int r = 0; r < kRvRows; ++r) {
@@ -169,9 +187,9 @@ __device__ __forceinline__ void rv_rows(const Src& src, int rows, int chunks, co
     for (int d = 0; d < kRvAhead; ++d)
 #pragma unroll
       for (int r = 0; r < kRvRows; ++r) ahead[d][r] = ahead[d + 1][r];
-    rv_load(src, pre, rows, chunks, ahead[kRvAhead]);
-    pre.next(nc);
-    if (cur.ci == nc - 1) {
+    rv_load(src, t, pre, rows, ahead[kRvAhead]);
+    pre.next(t);
+    if (cur.ci == t.nc - 1) {
       // lanes 0 / 8 / 16 / 24 end up with the sums of rows 0 / 1 / 2 / 3
       const bool up16 = lane & 16, up8 = lane & 8;
       float a0 = (up16 ? acc[2] : acc[0]) + __shfl_xor_sync(0xffffffffu, up16 ? acc[0] : acc[2], 16);
@@ -179,19 +197,22 @@ __device__ __forceinline__ void rv_rows(const Src& src, int rows, int chunks, co
       float b = (up8 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, up8 ? a0 : a1, 8);
 #pragma unroll
       for (int o = 4; o > 0; o >>= 1) b += __shfl_xor_sync(0xffffffffu, b, o);
-      if ((lane & 7) == 0) part[(cur.group * kRvRows + (lane >> 3)) * kRvWarps + warp] = b;
+      if ((lane & 7) == 0) part[(cur.group * kRvRows + (lane >> 3)) * kRvWarps + t.warp] = b;
 #pragma unroll
       for (int r = 0; r < kRvRows; ++r) acc[r] = 0.f;
     }
-    cur.next(nc);
+    cur.next(t);
   }
 }
 
-__device__ __forceinline__ float rv_total(const float* part, int row) {
-  const float4* q = reinterpret_cast<const float4*>(part + row * kRvWarps);
+__device__ __forceinline__ float rv_total(const RvTeam& t, const float* part, int row) {
   float s = 0.f;
-#pragma unroll
-  for (int i = 0; i < kRvWarps / 4; ++i) s += (q[i].x + q[i].y) + (q[i].z + q[i].w);
+  if (t.warps >= 4) {
+    const float4* q = reinterpret_cast<const float4*>(part + row * kRvWarps);
+    for (int i = 0; i < t.warps / 4; ++i) s += (q[i].x + q[i].y) + (q[i].z + q[i].w);
+  } else {
+    for (int i = 0; i < t.warps; ++i) s += part[row * kRvWarps + i];
+  }
   return s;
 }
 
@@ -220,24 +241,24 @@ __global__ void __launch_bounds__(kRvThreads, 1) rv_dense_kernel(const RvDensePa
   const RvVec v{smem + kRvBatchRows * kRvWarps, smem + kRvBatchRows * kRvWarps + rv_half_words(kp)};
   const int r0 = static_cast<int>(static_cast<long long>(p.n) * blockIdx.x / gridDim.x);
   const int r1 = static_cast<int>(static_cast<long long>(p.n) * (blockIdx.x + 1) / gridDim.x);
-  const int nc = (kp / 8 + kRvThreads - 1) / kRvThreads;
+  const RvTeam team(kp / 8);
   uint4 ahead[kRvAhead + 1][kRvRows];
   {
     const RvDenseSrc src{p.w + r0 * p.ldw, p.ldw};
-    RvCursor c;
+    RvCursor c(team);
 #pragma unroll
     for (int d = 0; d <= kRvAhead; ++d) {
-      rv_load(src, c, min(r1 - r0, kRvBatchRows), kp / 8, ahead[d]);
-      c.next(nc);
+      rv_load(src, team, c, min(r1 - r0, kRvBatchRows), ahead[d]);
+      c.next(team);
     }
   }
   pdl_wait();
   rv_stage(p.in, v, red);
   for (int b = r0; b < r1; b += kRvBatchRows) {
     const int rows = min(r1 - b, kRvBatchRows);
-    rv_rows(RvDenseSrc{p.w + b * p.ldw, p.ldw}, rows, kp / 8, v, part, ahead, b == r0);
+    rv_rows(RvDenseSrc{p.w + b * p.ldw, p.ldw}, team, rows, v, part, ahead, b == r0);
     __syncthreads();
-    for (int i = threadIdx.x; i < rows; i += kRvThreads) p.out[b + i] = rv_total(part, i) + (p.bias != nullptr ? p.bias[b + i] : 0.f);
+    for (int i = threadIdx.x; i < rows; i += kRvThreads) p.out[b + i] = rv_total(team, part, i) + (p.bias != nullptr ? p.bias[b + i] : 0.f);
     __syncthreads();
   }
 }
@@ -287,6 +308,7 @@ __global__ void __launch_bounds__(kRvThreads, 1) rv_gate_up_kernel(const RvGateU
       }
   }
   __syncthreads();
+  const RvTeam team(kp / 8);
   const int n_feat = p.ff_sh + p.top * p.ff;
   const int f0 = static_cast<int>(static_cast<long long>(n_feat) * blockIdx.x / gridDim.x);
   const int f1 = static_cast<int>(static_cast<long long>(n_feat) * (blockIdx.x + 1) / gridDim.x);
@@ -303,14 +325,14 @@ __global__ void __launch_bounds__(kRvThreads, 1) rv_gate_up_kernel(const RvGateU
       }
     }
     __syncthreads();
-    rv_rows(RvPtrSrc{s_row}, 2 * feats, kp / 8, v, part, ahead, false);
+    rv_rows(RvPtrSrc{s_row}, team, 2 * feats, v, part, ahead, false);
     __syncthreads();
     for (int i = threadIdx.x; i < feats; i += kRvThreads) {
       const int f = b + i;
       const bool shared = f < p.ff_sh;
       const int j = shared ? 0 : (f - p.ff_sh) / p.ff;
       const int dst = shared ? f : pad_to(p.ff_sh, 8) + j * pad_to(p.ff, 8) + (f - p.ff_sh) - j * p.ff;
-      p.hidden[dst] = clamped_gate(rv_total(part, 2 * i), rv_total(part, 2 * i + 1), shared ? p.limit_sh : p.limit, p.alpha);
+      p.hidden[dst] = clamped_gate(rv_total(team, part, 2 * i), rv_total(team, part, 2 * i + 1), shared ? p.limit_sh : p.limit, p.alpha);
     }
     __syncthreads();
   }
@@ -363,12 +385,13 @@ __global__ void __launch_bounds__(kRvThreads, 1) rv_down_kernel(const RvDownPara
   __syncthreads();
   const int r0 = static_cast<int>(static_cast<long long>(p.dim) * blockIdx.x / gridDim.x);
   const int r1 = static_cast<int>(static_cast<long long>(p.dim) * (blockIdx.x + 1) / gridDim.x);
+  const RvTeam team(kp / 8);
   uint4 ahead[kRvAhead + 1][kRvRows];
   for (int b = r0; b < r1; b += kRvBatchRows) {
     const int rows = min(r1 - b, kRvBatchRows);
-    rv_rows(RvPieceSrc{pieces, b}, rows, kp / 8, v, part, ahead, false);
+    rv_rows(RvPieceSrc{pieces, b}, team, rows, v, part, ahead, false);
     __syncthreads();
-    for (int i = threadIdx.x; i < rows; i += kRvThreads) p.out[b + i] = rv_total(part, i);
+    for (int i = threadIdx.x; i < rows; i += kRvThreads) p.out[b + i] = rv_total(team, part, i);
     __syncthreads();
   }
 }

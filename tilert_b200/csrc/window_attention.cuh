@@ -50,6 +50,22 @@ __device__ __forceinline__ float mixed_value(const QkvPrep& p, const QkvShape& s
   return v;
 }
 
+// This thread's share of the sum of squares of row[0..n).
+__device__ __forceinline__ float sum_squares(const float* row, int n) {
+  float s = 0.f;
+  if (n % 4 == 0 && reinterpret_cast<uintptr_t>(row) % 16 == 0) {
+    const float4* r4 = reinterpret_cast<const float4*>(row);
+#pragma unroll 4
+    for (int i = threadIdx.x; i < n / 4; i += blockDim.x) {
+      const float4 v = r4[i];
+      s += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) s += row[i] * row[i];
+  }
+  return s;
+}
+
 __device__ __forceinline__ float rinv_of(float sum, int n, float eps) { return 1.f / sqrtf(sum / static_cast<float>(n) + eps); }
 
 // ------------------------------------------------------------------ a portion of tokens: prepare
@@ -71,9 +87,7 @@ __global__ void __launch_bounds__(256) qkv_rows_kernel(const QkvRowsParams a) {
   const int t = blockIdx.x;
   const float* row = a.p.qkv + t * a.p.ld;
   const int nq = s.heads * s.dim, nk = s.kv_heads * s.dim, nv = s.kv_heads * s.vdim;
-  float sq = 0.f, sk = 0.f;
-  for (int i = threadIdx.x; i < nq; i += 256) sq += row[i] * row[i];
-  for (int i = threadIdx.x; i < nk; i += 256) sk += row[nq + i] * row[nq + i];
+  const float sq = sum_squares(row, nq), sk = sum_squares(row + nq, nk);
   const float rq = rinv_of(cta_sum(sq, red), nq, a.p.eps), rk = rinv_of(cta_sum(sk, red), nk, a.p.eps);
   const long long slot = (*a.pos + t) % s.ring;
   T* q = reinterpret_cast<T*>(a.q) + static_cast<long long>(t) * s.heads * s.dimp;
@@ -117,6 +131,32 @@ __host__ __device__ inline size_t attn_rows_smem(int dimp, int vdimp) {
   return (kAttnHeads * dimp + kAttnHeads * kAttnChunk + kAttnThreads * kAttnHeads * 8) * sizeof(float);
 }
 
+// Key range of one part of a query at `pos`.
+struct KeyRange {
+  int lo, hi;
+};
+__device__ __forceinline__ KeyRange key_range(int pos, int window, int n_splits, int split) {
+  const int first = window > 0 ? max(0, pos - window + 1) : 0;
+  const int per = (pos + 1 - first + n_splits - 1) / n_splits;
+  const int lo = min(first + split * per, pos + 1);
+  return {lo, min(lo + per, pos + 1)};
+}
+
+// Requests the part's cached rows into the L2 before the launch may read anything (a hint: what it reads of the
+// position may be old, the addresses stay inside the cache either way).
+template <typename T>
+__device__ __forceinline__ void prefetch_range(const AttnRowsParams& a, int g) {
+  const QkvShape& s = a.s;
+  const KeyRange r = key_range(max(*reinterpret_cast<const volatile int*>(a.pos), 0), s.window, a.n_splits, blockIdx.x);
+  for (int key = r.lo + static_cast<int>(threadIdx.x); key < r.hi; key += kAttnThreads) {
+    const long long row = static_cast<long long>(g) * s.ring + key % s.ring;
+    const char* k = reinterpret_cast<const char*>(reinterpret_cast<const T*>(a.k_cache) + row * s.dimp);
+    const char* v = reinterpret_cast<const char*>(reinterpret_cast<const T*>(a.v_cache) + row * s.vdimp);
+    for (int b = 0; b < s.dimp * static_cast<int>(sizeof(T)); b += 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(k + b));
+    for (int b = 0; b < s.vdimp * static_cast<int>(sizeof(T)); b += 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(v + b));
+  }
+}
+
 template <typename T, bool FUSED>
 __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsParams a) {
   extern __shared__ __align__(16) float smem[];
@@ -124,9 +164,10 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
   __shared__ float s_m[kAttnHeads], s_l[kAttnHeads], s_corr[kAttnHeads];
   __shared__ int s_last;
   pdl_launch_dependents();
-  pdl_wait();
   const QkvShape& s = a.s;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (FUSED) prefetch_range<T>(a, blockIdx.y / ((s.heads / s.kv_heads + kAttnHeads - 1) / kAttnHeads));
+  pdl_wait();
   const int group = s.heads / s.kv_heads, n_hb = (group + kAttnHeads - 1) / kAttnHeads;
   const int split = blockIdx.x, g = blockIdx.y / n_hb, hb = blockIdx.y - g * n_hb, t = blockIdx.z;
   const int h0 = g * group + hb * kAttnHeads;
@@ -135,19 +176,15 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
   float* qs = smem;                               // [kAttnHeads][dimp], scaled
   float* sc = qs + kAttnHeads * s.dimp;           // [kAttnHeads][kAttnChunk]
   float* red2 = sc + kAttnHeads * kAttnChunk;     // [threads][kAttnHeads * 8]
-  const int first = s.window > 0 ? max(0, pos - s.window + 1) : 0;
-  const int n = pos + 1 - first;
-  const int per = (n + a.n_splits - 1) / a.n_splits;
-  const int lo = min(first + split * per, pos + 1), hi = min(lo + per, pos + 1);
+  const KeyRange range = key_range(pos, s.window, a.n_splits, split);
+  const int lo = range.lo, hi = range.hi;
   T* kc = reinterpret_cast<T*>(a.k_cache) + static_cast<long long>(g) * s.ring * s.dimp;
   T* vc = reinterpret_cast<T*>(a.v_cache) + static_cast<long long>(g) * s.ring * s.vdimp;
 
   if (FUSED) {
     const int nq = s.heads * s.dim, nk = s.kv_heads * s.dim;
     const float* row = a.p.qkv;
-    float sq = 0.f, sk = 0.f;
-    for (int i = tid; i < nq; i += kAttnThreads) sq += row[i] * row[i];
-    for (int i = tid; i < nk; i += kAttnThreads) sk += row[nq + i] * row[nq + i];
+    const float sq = sum_squares(row, nq), sk = sum_squares(row + nq, nk);
     const float rq = rinv_of(cta_sum(sq, red), nq, a.p.eps), rk = rinv_of(cta_sum(sk, red), nk, a.p.eps);
     for (int i = tid; i < kAttnHeads * s.dimp; i += kAttnThreads) {
       const int h = i / s.dimp, d = i - h * s.dimp;
@@ -187,7 +224,8 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
   for (int c0 = lo; c0 < hi; c0 += kAttnChunk) {
     const int cn = min(kAttnChunk, hi - c0), slot0 = c0 % s.ring;
     // scores: eight lanes per key, four keys per warp and step
-    for (int k0 = warp * 4; k0 < kAttnChunk; k0 += kAttnThreads / 8) {
+    const int cn32 = pad_to(cn, 32);
+    for (int k0 = warp * 4; k0 < cn32; k0 += kAttnThreads / 8) {
       const int key = k0 + (lane >> 3);
       float d[kAttnHeads];
 #pragma unroll
@@ -216,10 +254,10 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
     __syncthreads();
     if (warp < kAttnHeads) {
       float m = -INFINITY;
-      for (int i = lane; i < kAttnChunk; i += 32) m = fmaxf(m, sc[warp * kAttnChunk + i]);
+      for (int i = lane; i < cn32; i += 32) m = fmaxf(m, sc[warp * kAttnChunk + i]);
       m = fmaxf(warp_max(m), s_m[warp]);
       float l = 0.f;
-      for (int i = lane; i < kAttnChunk; i += 32) {
+      for (int i = lane; i < cn32; i += 32) {
         const float e = expf(sc[warp * kAttnChunk + i] - m);
         sc[warp * kAttnChunk + i] = e;
         l += e;
@@ -293,28 +331,41 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
   __syncthreads();
   if (!s_last) return;
   __threadfence();
+  // weight of every part, one warp per head: exp(max - overall max), and the overall sum (red2 is free again)
+  float* wgt = red2;  // [kAttnHeads][n_splits]
+  if (warp < nh) {
+    const float* mh = ml + static_cast<long long>(h0 + warp) * a.n_splits * 2;
+    float m = -INFINITY, l = 0.f;
+    for (int k = lane; k < a.n_splits; k += 32) m = fmaxf(m, __ldcg(mh + 2 * k));
+    m = warp_max(m);
+    for (int k = lane; k < a.n_splits; k += 32) {
+      const float c = expf(__ldcg(mh + 2 * k) - m);  // an empty part has max -inf: weight 0
+      wgt[warp * a.n_splits + k] = c;
+      l += c * __ldcg(mh + 2 * k + 1);
+    }
+    l = warp_sum(l);
+    if (lane == 0) s_l[warp] = l;
+  }
+  __syncthreads();
   for (int i = tid; i < nh * s.vdim; i += kAttnThreads) {
     const int h = i / s.vdim, v = i - h * s.vdim;
-    const float* mh = ml + (h0 + h) * a.n_splits * 2;
-    float m = -INFINITY;
-    for (int k = 0; k < a.n_splits; ++k) m = fmaxf(m, __ldcg(mh + 2 * k));
-    float o = 0.f, l = 0.f;
-    for (int k = 0; k < a.n_splits; ++k) {
-      const float c = expf(__ldcg(mh + 2 * k) - m);  // an empty part has max -inf: weight 0
-      l += c * __ldcg(mh + 2 * k + 1);
-      o += c * __ldcg(a.part + (static_cast<long long>(h0 + h) * a.n_splits + k) * s.vdimp + v);
-    }
+    const float* src = a.part + static_cast<long long>(h0 + h) * a.n_splits * s.vdimp + v;
+    const float* w = wgt + h * a.n_splits;
+    float o = 0.f;
+#pragma unroll 8
+    for (int k = 0; k < a.n_splits; ++k) o += w[k] * __ldcg(src + static_cast<long long>(k) * s.vdimp);
     const long long dst = t * a.ldo + (h0 + h) * s.vdim + v;
     if (FUSED)
-      reinterpret_cast<float*>(a.out)[dst] = o / l;
+      reinterpret_cast<float*>(a.out)[dst] = o / s_l[h];
     else
-      act_st(reinterpret_cast<T*>(a.out) + dst, o / l);
+      act_st(reinterpret_cast<T*>(a.out) + dst, o / s_l[h]);
   }
 }
 
 // ------------------------------------------------------------------ a portion of tokens, bf16 tensor-core tiles
 // 64 rows per CTA = (tokens x query heads of one key/value head), so the heads of a group share the key tiles.
-// 64 keys per tile, two tiles in flight (cp.async); four warps of 16 rows; online softmax in registers.
+// 64 keys per tile; the next keys are requested (cp.async) before a tile's scores, the next values after its product;
+// four warps of 16 rows, three CTAs per SM at 128-wide heads; online softmax in registers.
 constexpr int kFaRows = 64, kFaKeys = 64, kFaThreads = 128;
 constexpr int kFaMaxHeads = 16;  // query heads of a group per CTA
 
@@ -331,7 +382,7 @@ struct AttnPrefillParams {
 };
 
 __host__ __device__ inline size_t attn_prefill_smem(int dimp, int vdimp) {
-  return (static_cast<size_t>(kFaRows + 2 * kFaKeys) * (dimp + 8) + 2 * kFaKeys * (vdimp + 8)) * 2;
+  return (static_cast<size_t>(kFaRows + 2 * kFaKeys) * (dimp + 8) + kFaKeys * (vdimp + 8)) * 2;
 }
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
@@ -343,7 +394,7 @@ __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_gr
 
 // DV16: value tiles of 16 columns the accumulator has room for (vdimp <= 16 * DV16)
 template <int DV16>
-__global__ void __launch_bounds__(kFaThreads) attn_prefill_kernel(const AttnPrefillParams a) {
+__global__ void __launch_bounds__(kFaThreads, DV16 <= 8 ? 3 : 1) attn_prefill_kernel(const AttnPrefillParams a) {
   extern __shared__ __align__(16) __nv_bfloat16 fsm[];
   pdl_launch_dependents();
   pdl_wait();
@@ -365,7 +416,7 @@ __global__ void __launch_bounds__(kFaThreads) attn_prefill_kernel(const AttnPref
   const __nv_bfloat16* vc = a.v_cache + static_cast<long long>(g) * s.ring * s.vdimp;
   const int lo = s.window > 0 ? max(0, pos0 + t0 - s.window + 1) : 0, hi = pos0 + t0 + nt;  // keys any row sees
 
-  const int dch = s.dimp / 8, vch = s.vdimp / 8;
+  const int dch = s.dimp / 8;
   for (int i = tid; i < kFaRows * dch; i += kFaThreads) {
     const int r = i / dch, c = i - r * dch;
     const int tt = r / hpb, h = r - tt * hpb;
@@ -373,25 +424,18 @@ __global__ void __launch_bounds__(kFaThreads) attn_prefill_kernel(const AttnPref
     const long long row = ok ? static_cast<long long>(t0 + tt) * s.heads + h0 + h : 0;
     cp_async16(qs + r * qp + c * 8, a.q + row * s.dimp + c * 8, ok);
   }
-  auto load_tile = [&](int k0, int buf) {
-    __nv_bfloat16* kd = ks + buf * kFaKeys * qp;
-    __nv_bfloat16* vd = vs + buf * kFaKeys * vpitch;
-    const int slot0 = k0 % s.ring;
-    for (int i = tid; i < kFaKeys * dch; i += kFaThreads) {
-      const int r = i / dch, c = i - r * dch;
+  auto load_rows = [&](__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int width, int k0) {
+    const int ch = width / 8, slot0 = k0 % s.ring;
+    for (int i = tid; i < kFaKeys * ch; i += kFaThreads) {
+      const int r = i / ch, c = i - r * ch;
       const bool ok = k0 + r < hi;
       const long long slot = ok ? slot0 + r - (slot0 + r >= s.ring ? s.ring : 0) : 0;
-      cp_async16(kd + r * qp + c * 8, kc + slot * s.dimp + c * 8, ok);
-    }
-    for (int i = tid; i < kFaKeys * vch; i += kFaThreads) {
-      const int r = i / vch, c = i - r * vch;
-      const bool ok = k0 + r < hi;
-      const long long slot = ok ? slot0 + r - (slot0 + r >= s.ring ? s.ring : 0) : 0;
-      cp_async16(vd + r * vpitch + c * 8, vc + slot * s.vdimp + c * 8, ok);
+      cp_async16(dst + r * pitch + c * 8, src + slot * width + c * 8, ok);
     }
     cp_async_commit();
   };
-  load_tile(lo, 0);
+  load_rows(ks, qp, kc, s.dimp, lo);
+  load_rows(vs, vpitch, vc, s.vdimp, lo);
 
   float o[DV16 * 2][4];
 #pragma unroll
@@ -410,15 +454,11 @@ __global__ void __launch_bounds__(kFaThreads) attn_prefill_kernel(const AttnPref
   const int n_tiles = (hi - lo + kFaKeys - 1) / kFaKeys;
   for (int tile = 0; tile < n_tiles; ++tile) {
     const int k0 = lo + tile * kFaKeys, buf = tile & 1;
-    if (tile + 1 < n_tiles) {
-      load_tile(k0 + kFaKeys, buf ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
+    const bool more = tile + 1 < n_tiles;
+    cp_async_wait<1>();  // all but the newest group: this tile's keys (its values are the newest)
     __syncthreads();
+    if (more) load_rows(ks + (buf ^ 1) * kFaKeys * qp, qp, kc, s.dimp, k0 + kFaKeys);
     const __nv_bfloat16* kt = ks + buf * kFaKeys * qp;
-    const __nv_bfloat16* vt = vs + buf * kFaKeys * vpitch;
     float sacc[8][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i)
@@ -437,15 +477,27 @@ __global__ void __launch_bounds__(kFaThreads) attn_prefill_kernel(const AttnPref
       }
     }
     float mx[2] = {-INFINITY, -INFINITY};
+    // every key of an inner tile is visible to every row (rows without a token are never stored)
+    const bool inner = k0 + kFaKeys - 1 <= pos0 + t0 && hi - 1 - k0 < win;
+    if (inner) {
 #pragma unroll
-    for (int nt8 = 0; nt8 < 8; ++nt8)
+      for (int nt8 = 0; nt8 < 8; ++nt8)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int kpos = k0 + nt8 * 8 + (lane & 3) * 2 + (j & 1), i = j >> 1;
-        const bool ok = kpos <= qpos[i] && qpos[i] - kpos < win;
-        sacc[nt8][j] = ok ? sacc[nt8][j] * a.scale : -INFINITY;
-        mx[i] = fmaxf(mx[i], sacc[nt8][j]);
-      }
+        for (int j = 0; j < 4; ++j) {
+          sacc[nt8][j] *= a.scale;
+          mx[j >> 1] = fmaxf(mx[j >> 1], sacc[nt8][j]);
+        }
+    } else {
+#pragma unroll
+      for (int nt8 = 0; nt8 < 8; ++nt8)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int kpos = k0 + nt8 * 8 + (lane & 3) * 2 + (j & 1), i = j >> 1;
+          const bool ok = kpos <= qpos[i] && qpos[i] - kpos < win;
+          sacc[nt8][j] = ok ? sacc[nt8][j] * a.scale : -INFINITY;
+          mx[i] = fmaxf(mx[i], sacc[nt8][j]);
+        }
+    }
     float corr[2], msafe[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -481,13 +533,15 @@ __global__ void __launch_bounds__(kFaThreads) attn_prefill_kernel(const AttnPref
       pa[nb][2] = pack_bf16x2(e[4], e[5]);
       pa[nb][3] = pack_bf16x2(e[6], e[7]);
     }
+    if (more) cp_async_wait<1>(); else cp_async_wait<0>();  // this tile's values
+    __syncthreads();
 #pragma unroll
     for (int vb = 0; vb < DV16; ++vb) {
       if (vb * 16 < s.vdimp) {
 #pragma unroll
         for (int nb = 0; nb < 4; ++nb) {
           uint32_t bv[4];  // keys 0-7 / 8-15 of columns 0-7, then of columns 8-15
-          ldmatrix_x4_trans(bv, vt + (nb * 16 + (lane & 15)) * vpitch + vb * 16 + (lane >> 4) * 8);
+          ldmatrix_x4_trans(bv, vs + (nb * 16 + (lane & 15)) * vpitch + vb * 16 + (lane >> 4) * 8);
           const uint32_t b0[2] = {bv[0], bv[1]}, b1[2] = {bv[2], bv[3]};
           mma_bf16_16816(o[vb * 2], pa[nb], b0);
           mma_bf16_16816(o[vb * 2 + 1], pa[nb], b1);
@@ -495,6 +549,7 @@ __global__ void __launch_bounds__(kFaThreads) attn_prefill_kernel(const AttnPref
       }
     }
     __syncthreads();
+    if (more) load_rows(vs, vpitch, vc, s.vdimp, k0 + kFaKeys);
   }
 #pragma unroll
   for (int i = 0; i < 2; ++i) {

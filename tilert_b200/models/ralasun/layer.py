@@ -146,7 +146,7 @@ class RalasunLayer:
         self.cache = RingKVCache(m.kv_heads, m.dim, m.vdim, m.window, args.max_seq_len, portion, device, dtype)
         self.n_q, self.n_kv = m.heads * m.dim, m.kv_heads * (m.dim + m.vdim)
         self.head_blocks = ops.head_blocks(m.heads, m.kv_heads)
-        self.max_splits = max(1, 2 * ops.num_sms(device) // self.head_blocks)
+        self.max_splits = max(1, 2 * ops.num_sms(device) // self.head_blocks)  # (two thread blocks per SM)
 
     def _v_first(self, rows: int):
         """Values of the first mixing layer, [rows, kv_heads * vdim] (all mixing layers agree on the size)."""
