@@ -21,7 +21,7 @@ def rms(x: torch.Tensor, eps: float) -> torch.Tensor:
 
 
 def norm_around_one(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
-    """RMS norm whose gain is 1 + w (the weight is stored around zero)."""
+    """RMS norm whose gain is 1 + w."""
     return rms(x, eps) * (1 + w)
 
 
@@ -36,7 +36,7 @@ def visible(i: int, size: int | None) -> range:
 
 
 def mix_values(v: torch.Tensor, first: torch.Tensor, lam: float) -> torch.Tensor:
-    """A layer's values pulled towards the first mixing layer's values of the same token."""
+    """A layer's values pulled towards those of the first mixing layer, position by position."""
     return (1 - lam) * v + lam * first
 
 

@@ -208,14 +208,14 @@ extern "C" int tilert_gqa_gemm_op(TgContext* ctx, const void* x, long long ldx, 
   }
   const long long w_rows = static_cast<long long>(n_groups > 0 ? n_groups : 1) * per * n;
   const int ft = (n + 127) / 128;
-  // Token tile: waves of tiles over the SMs times the relative cost of a tile (narrow tiles reuse a weight tile less).
-  // Groups are taken as equally long, each ending in a half-filled tile.
+  // Token tile.  One weight: waves of tiles over the SMs times the relative cost of a tile (a narrow tile moves more
+  // bytes per product through the L2).  Groups: the widest tile that an average group nearly fills.
   auto cost = [&](int bn, double tile) {
-    const double tiles = n_groups > 0 ? ft * (static_cast<double>(rows) / bn + 0.5 * n_groups) : static_cast<double>(ft) * ((rows + bn - 1) / bn);
-    return std::ceil(tiles / ctx->num_sms) * tile;
+    if (n_groups > 0) return bn == 64 || rows / n_groups >= bn * 3 / 4 ? 1.0 / bn : 1.0;
+    return std::ceil(static_cast<double>(ft) * ((rows + bn - 1) / bn) / ctx->num_sms) * tile;
   };
   if (gated) return cost(128, 1.0) <= cost(64, 0.6) ? launch_tc<128, true>(ctx, p, w_rows, stream) : launch_tc<64, true>(ctx, p, w_rows, stream);
-  const double c256 = cost(256, 1.0), c128 = cost(128, 0.56), c64 = cost(64, 0.34);
+  const double c256 = cost(256, 1.0), c128 = cost(128, 0.75), c64 = cost(64, 0.55);
   if (c256 <= c128 && c256 <= c64) return launch_tc<256, false>(ctx, p, w_rows, stream);
   if (c128 <= c64) return launch_tc<128, false>(ctx, p, w_rows, stream);
   return launch_tc<64, false>(ctx, p, w_rows, stream);

@@ -1,6 +1,6 @@
 // Row kernels around the norms of a residual stream kept in f32: embedding + norm, sublayer output -> norm ->
 // residual, and the norm in front of the vocabulary head.  One CTA per token; the gain vectors are f32 and already
-// hold the factor the norm multiplies with (a weight stored around zero arrives as 1 + w).
+// hold the factor the norm multiplies with (a weight that is an offset from one arrives as 1 + w).
 #pragma once
 
 #include "act.cuh"

@@ -4,8 +4,8 @@
 // the positions j with 0 <= i - j < window (window 0: every j <= i); the ring has to hold the window of the oldest
 // query of a launch together with every position of the launch.  Rows are padded to 16 elements with zeros.
 //
-// Queries and keys are RMS-normalised over their whole projection (all heads at once) before they are split into
-// heads; values can be mixed with the values an earlier layer had for the same token.  Both happen here:
+// Queries and keys are RMS-normalised over their whole projection, one statistic for all heads; values can be blended
+// with what an earlier layer computed at that position.  Both happen here:
 //   qkv_rows_kernel          a portion of tokens: normalised queries out, keys and values into the ring
 //   attn_prefill_kernel      a portion of tokens, bf16 tensor-core tiles with an online softmax
 //   attn_rows_kernel<T, true>   one token: the preparation, the cache write and the attention in one launch, the
@@ -111,6 +111,9 @@ __global__ void __launch_bounds__(256) qkv_rows_kernel(const QkvRowsParams a) {
 constexpr int kAttnThreads = 256;
 constexpr int kAttnHeads = 4;    // query heads per CTA
 constexpr int kAttnChunk = 128;  // keys per softmax step
+constexpr int kAttnPasses = kAttnChunk / 32;
+constexpr int kAttnAhead = 4;    // value rows a thread loads together
+static_assert(kAttnThreads == 256, "eight warps of four keys make a pass of 32");
 
 struct AttnRowsParams {
   QkvShape s;
@@ -223,33 +226,47 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
   // the keys of a launch lie in fewer than `ring` consecutive positions, so one subtraction wraps a row index
   for (int c0 = lo; c0 < hi; c0 += kAttnChunk) {
     const int cn = min(kAttnChunk, hi - c0), slot0 = c0 % s.ring;
-    // scores: eight lanes per key, four keys per warp and step
+    // scores: eight lanes per key, four keys per warp and pass; the passes' keys are loaded together
     const int cn32 = pad_to(cn, 32);
-    for (int k0 = warp * 4; k0 < cn32; k0 += kAttnThreads / 8) {
-      const int key = k0 + (lane >> 3);
-      float d[kAttnHeads];
+    {
+      const T* kr[kAttnPasses];
+      float d[kAttnPasses][kAttnHeads];
 #pragma unroll
-      for (int h = 0; h < kAttnHeads; ++h) d[h] = 0.f;
-      if (key < cn) {
+      for (int it = 0; it < kAttnPasses; ++it) {
+        const int key = min(it * 32 + warp * 4 + (lane >> 3), cn - 1);  // past the end: the last key, dropped below
         const int slot = slot0 + key - (slot0 + key >= s.ring ? s.ring : 0);
-        const T* kr = kc + static_cast<long long>(slot) * s.dimp;
-        for (int c = lane & 7; c < s.dimp / 8; c += 8) {
-          float f[8];
-          act_ld8(kr + c * 8, f);
+        kr[it] = kc + static_cast<long long>(slot) * s.dimp;
 #pragma unroll
-          for (int h = 0; h < kAttnHeads; ++h) {
-            const float4 q0 = *reinterpret_cast<const float4*>(qs + h * s.dimp + c * 8);
-            const float4 q1 = *reinterpret_cast<const float4*>(qs + h * s.dimp + c * 8 + 4);
-            d[h] += f[0] * q0.x + f[1] * q0.y + f[2] * q0.z + f[3] * q0.w + f[4] * q1.x + f[5] * q1.y + f[6] * q1.z + f[7] * q1.w;
-          }
+        for (int h = 0; h < kAttnHeads; ++h) d[it][h] = 0.f;
+      }
+#pragma unroll 2
+      for (int c = lane & 7; c < s.dimp / 8; c += 8) {
+        float f[kAttnPasses][8];
+#pragma unroll
+        for (int it = 0; it < kAttnPasses; ++it)
+          if (it * 32 < cn) act_ld8(kr[it] + c * 8, f[it]);
+#pragma unroll
+        for (int h = 0; h < kAttnHeads; ++h) {
+          const float4 q0 = *reinterpret_cast<const float4*>(qs + h * s.dimp + c * 8);
+          const float4 q1 = *reinterpret_cast<const float4*>(qs + h * s.dimp + c * 8 + 4);
+#pragma unroll
+          for (int it = 0; it < kAttnPasses; ++it)
+            if (it * 32 < cn)
+              d[it][h] += f[it][0] * q0.x + f[it][1] * q0.y + f[it][2] * q0.z + f[it][3] * q0.w + f[it][4] * q1.x + f[it][5] * q1.y +
+                          f[it][6] * q1.z + f[it][7] * q1.w;
         }
       }
 #pragma unroll
-      for (int h = 0; h < kAttnHeads; ++h) {
+      for (int it = 0; it < kAttnPasses; ++it)
+        if (it * 32 < cn) {
+          const int key = it * 32 + warp * 4 + (lane >> 3);
 #pragma unroll
-        for (int o = 4; o > 0; o >>= 1) d[h] += __shfl_xor_sync(0xffffffffu, d[h], o);
-        if ((lane & 7) == 0) sc[h * kAttnChunk + key] = key < cn ? d[h] : -INFINITY;
-      }
+          for (int h = 0; h < kAttnHeads; ++h) {
+#pragma unroll
+            for (int o = 4; o > 0; o >>= 1) d[it][h] += __shfl_xor_sync(0xffffffffu, d[it][h], o);
+            if ((lane & 7) == 0) sc[h * kAttnChunk + key] = key < cn ? d[it][h] : -INFINITY;
+          }
+        }
     }
     __syncthreads();
     if (warp < kAttnHeads) {
@@ -276,15 +293,23 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
       for (int h = 0; h < kAttnHeads; ++h)
 #pragma unroll
         for (int j = 0; j < 8; ++j) acc[h][j] *= s_corr[h];
-      for (int key = kl; key < cn; key += key_lanes) {
-        float f[8];
-        const int slot = slot0 + key - (slot0 + key >= s.ring ? s.ring : 0);
-        act_ld8(vc + static_cast<long long>(slot) * s.vdimp + vp * 8, f);
+      for (int k0 = kl; k0 < cn; k0 += kAttnAhead * key_lanes) {
+        float f[kAttnAhead][8];
 #pragma unroll
-        for (int h = 0; h < kAttnHeads; ++h) {
-          const float w = sc[h * kAttnChunk + key];
+        for (int u = 0; u < kAttnAhead; ++u) {
+          const int key = min(k0 + u * key_lanes, cn - 1);
+          const int slot = slot0 + key - (slot0 + key >= s.ring ? s.ring : 0);
+          act_ld8(vc + static_cast<long long>(slot) * s.vdimp + vp * 8, f[u]);
+        }
 #pragma unroll
-          for (int j = 0; j < 8; ++j) acc[h][j] += w * f[j];
+        for (int u = 0; u < kAttnAhead; ++u) {
+          const int key = k0 + u * key_lanes;
+#pragma unroll
+          for (int h = 0; h < kAttnHeads; ++h) {
+            const float w = key < cn ? sc[h * kAttnChunk + key] : 0.f;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) acc[h][j] += w * f[u][j];
+          }
         }
       }
     }

@@ -31,7 +31,7 @@ def padded_rows(w: torch.Tensor, device) -> torch.Tensor:
 
 
 def one_plus(w: torch.Tensor, device) -> torch.Tensor:
-    """f32 gain of a norm whose weight is stored around zero, zeros beyond its length."""
+    """f32 gain of a norm whose weight is an offset from one, zeros beyond its length."""
     g = 1.0 + w.to(device, F32)
     return torch.nn.functional.pad(g, (0, pad(g.numel()) - g.numel())).contiguous()
 

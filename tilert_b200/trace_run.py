@@ -1,15 +1,16 @@
-"""Replays a trace of given token ids through a model, step by step, and writes the logits that are asked for.
+"""Replays recorded token ids: every request's tokens go through a model in the steps of the recording, and the logits
+at the places a step names are written out.  Nothing is sampled.
 
-    bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR [--max-tokens N]
+    bin/trace_run --model MODEL_DIR --out LOGITS_DIR [--dtype float32] [--max-tokens N] < steps.jsonl
 
-Standard input holds one JSON object per line,
+A step is one line of JSON,
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["a"]}
+    {"step": 7, "entries": [{"id": "chat-1", "tokens": [11, 12], "want": [1]}], "end": ["chat-1"]}
 
-and every step's wanted logits go to OUT/<step>.f32 (little-endian f32, [wanted, vocab]); "done <step>" is printed when a
-step has been run.  Nothing is sampled.  The model runs one sequence at a time: a request's tokens continue where its
-last step ended, and a new request may begin once the one before it has been ended.  Exit code 3: the model does not
-run in the asked-for type.
+where ``want`` holds indices into ``tokens`` and ``end`` names requests that are over.  LOGITS_DIR/7.f32 then holds the
+logits as raw little-endian f32 rows, and the line "done 7" follows.  The model runs one sequence at a time: a request
+continues where its previous step ended, and another may begin once it is over.  Exit code 3: the model's family does not
+run in the given type.
 """
 
 from __future__ import annotations
