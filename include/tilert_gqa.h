@@ -1,6 +1,6 @@
 /*
- * tilert_gqa -- C ABI of the grouped-query attention / mixture-of-experts path with bf16 weights: decoders whose
- * layers are q/k-normalised windowed attention with mixed values and clamped gated experts.
+ * tilert_gqa -- C ABI of decoders with bf16 weights: q/k-normalised windowed attention with mixed values or attention
+ * over a latent cache (windows, sinks, output gates), clamped gated units, dense or routed, RMS or layer norms.
  *
  * These are mechanisms, not a model: every size and constant is an argument.  Conventions are those of
  * tilert_b200.h: device pointers, caller-allocated outputs, asynchronous on `stream`, 0 or a negative TB_E* code,
@@ -14,7 +14,10 @@
  * logical length and the next multiple of 8 are zero.  f32 vectors of the one-token step are padded the same way.
  * Cache rows and prepared queries are padded to 16.
  *
- * Cache.  Keys [kv_heads, ring, dimp], values [kv_heads, ring, vdimp]; position p is row p % ring.
+ * Cache.  Keys [kv_heads, ring, dimp], values [kv_heads, ring, vdimp], or latent rows [ring, row] (see below); position
+ * p is row p % ring.
+ *
+ * Norms.  RMS norm, or the layer norm (mean taken off) where `centered` is set.  Biases of norms may be NULL.
  */
 #ifndef TILERT_GQA_H_
 #define TILERT_GQA_H_
@@ -45,27 +48,31 @@ int tilert_gqa_num_sms(TgContext* ctx);
 
 /* ---- norms on the residual stream ---- */
 
-/* x[t] = rms(table[tokens[t]]) * gain, also stored as activations in xh (may be NULL).  A token outside [0, vocab)
- * is refused on the device (status 4). */
+/* x[t] = rms(table[tokens[t]]) * gain (gain NULL: the row as it is), also stored as activations in xh (may be NULL).  A
+ * token outside [0, vocab) is refused on the device (status 4). */
 int tilert_gqa_embed_norm_op(TgContext* ctx, const long long* tokens, const void* table, long long ld_table, int vocab,
                              const float* gain, float eps, int rows, int dim, float* x, long long ldx, void* xh,
                              long long ldh, int f32, void* stream);
-/* x[t] += rms(y[t]) * gain, xh = x.  y is f32 [rows, ldy]; with y NULL the sublayer output is
- * sum_j slot_w[t, j] ye[slot_row[t, j]] (+ ysh[t] when given), the combine of a mixture of experts. */
+/* x[t] += norm(y[t]) (+ add), then xh = x, or its norm with gain2 (xh may be NULL without gain2).  y is f32 [rows, ldy];
+ * with y NULL and ye given the sublayer output is sum_j slot_w[t, j] ye[slot_row[t, j]] (+ ysh[t] when given), the
+ * combine of a mixture of experts; with both NULL (and gain NULL) there is none. */
 int tilert_gqa_residual_norm_op(TgContext* ctx, const float* y, long long ldy, const void* ye, long long lde,
                                 const int* slot_row, const float* slot_w, int top, const void* ysh, long long ldsh,
-                                const float* gain, float eps, int rows, int dim, float* x, long long ldx, void* xh,
-                                long long ldh, int f32, void* stream);
-/* out[i] = rms(x[rows[i]]) * gain */
+                                const float* gain, const float* bias, const float* add, const float* gain2,
+                                const float* bias2, int centered, float eps, int rows, int dim, float* x, long long ldx,
+                                void* xh, long long ldh, int f32, void* stream);
+/* out[i] = norm(x[rows[i]]) */
 int tilert_gqa_gather_norm_op(TgContext* ctx, const float* x, long long ldx, const int* rows, int n, const float* gain,
-                              float eps, int dim, void* out, long long ldo, int f32, void* stream);
+                              const float* bias, int centered, float eps, int dim, void* out, long long ldo, int f32,
+                              void* stream);
 
 /* ---- products of a portion of tokens ---- */
 
 /* out[t, :] = W x[t] (+ bias), W [n, ldw]; tensor cores (tcgen05) on bf16 rows, SIMT f32 otherwise.
  * out_f32: f32 output also from bf16 rows.  gated: W holds n gate rows, then n up rows, and
  * out = g / (1 + exp(-alpha g)) * (u + 1) with g = min(gate, limit), u = up within +-limit.
- * n_groups > 0: W is [n_groups][n or 2 n][ldw], counts[g] (device) rows of x and out belong to group g, in order. */
+ * n_groups > 0: W is [n_groups][n or 2 n][ldw], counts[g] (device) rows of x and out belong to group g, in order; with
+ * counts NULL every group has `rows` of them. */
 int tilert_gqa_gemm_op(TgContext* ctx, const void* x, long long ldx, int rows, const void* w, long long ldw, int n, int k,
                        int gated, float limit, float alpha, int n_groups, const int* counts, const float* bias, void* out,
                        long long ldo, int out_f32, int f32, void* stream);
@@ -98,10 +105,16 @@ int tilert_gqa_gather_rows_op(TgContext* ctx, const void* x, long long ldx, int 
 
 /* ---- one-token step ---- */
 
-/* v = x, or x + rms(y) * gain when y is given (stored to x_out when not NULL), or the norm of that with gain2;
- * out = W v (+ bias). */
-int tilert_gqa_vec_dense_op(TgContext* ctx, const float* x, const float* y, const float* gain, const float* gain2, float eps,
+/* v = x, or x + norm(y) when y is given, plus `add` when given (stored to x_out when not NULL), or the norm of that with
+ * gain2; out = W v (+ bias). */
+int tilert_gqa_vec_dense_op(TgContext* ctx, const float* x, const float* y, const float* gain, const float* norm_bias,
+                            const float* add, const float* gain2, const float* norm_bias2, int centered, float eps,
                             float* x_out, const void* w, long long ldw, const float* bias, int n, int k, float* out,
+                            void* stream);
+/* The same input into W [2][n][ldw] (gate rows, then up rows): out[n] as in gemm_op with `gated`. */
+int tilert_gqa_vec_gated_op(TgContext* ctx, const float* x, const float* y, const float* gain, const float* norm_bias,
+                            const float* add, const float* gain2, const float* norm_bias2, int centered, float eps,
+                            float* x_out, const void* w, long long ldw, int n, int k, float limit, float alpha, float* out,
                             void* stream);
 /* qkv_rows_op and attn_rows_op of one token at *pos in one launch.  n_splits CTAs share the keys of a head block; part
  * holds heads * n_splits * (vdimp + 2) floats, counter one zero word per head block.  out [heads * vdim] f32. */
@@ -120,6 +133,61 @@ int tilert_gqa_vec_gate_up_op(TgContext* ctx, const float* x, int dim, const flo
  * w_sh [dim][pad8(ff_sh)] or NULL. */
 int tilert_gqa_vec_down_op(TgContext* ctx, const float* hidden, const int* slot_ids, const float* slot_w, int top,
                            const void* w, const void* w_sh, int ff, int ff_sh, int dim, float* out, void* stream);
+
+/* ---- attention over a latent cache ---- */
+
+/* A cache row is [latent (rank), zero to rankp = pad16(rank) | rotated key part (rot), zero to row], row =
+ * pad32(rankp + rot); keys and values of all heads are linear in the latent, the rotated part is one for all heads.
+ * Projected queries hold per head ldh = pad8(dim) + pad8(rot) elements, the part to rotate at pad8(dim).
+ * Rotations.  Pairs (2i, 2i + 1) of the first rope_dims elements when interleaved, else (i, i + rope_dims / 2); rope is
+ * [positions][rope_dims], per position rope_dims / 2 cosines, then as many sines. */
+
+/* Elements of a cache row. */
+int tilert_gqa_latent_row_len(int rank, int rot);
+/* CTAs of latent_attn_op per part of the key range. */
+int tilert_gqa_latent_blocks(int heads, int tokens, int rank, int rot, int f32);
+/* Whether expanded_attn_op takes these sizes. */
+int tilert_gqa_expanded_fits(int dim, int rot, int vdim);
+/* From z [rows, ldz] f32 (query latent at 0, latent at off_c, key part at off_r): cq = rms(query latent) * q_gain, and
+ * the cache rows of positions *pos + t. */
+int tilert_gqa_latent_tokens_op(TgContext* ctx, const float* z, long long ldz, int q_rank, int off_c, int off_r,
+                                const float* q_gain, const float* c_gain, float eps, int rows, int rank, int rot,
+                                const float* rope, int positions, int rope_dims, int interleaved, const int* pos, int ring,
+                                void* cq, long long ldq, void* cache, int f32, void* stream);
+/* Projected queries [rows, ldq] f32, rotated.  lat NULL: out [rows, heads, pad16(dim) + pad16(rot)] (expanded form).  Else
+ * (absorbed form) the unrotated part to out [heads, rows, pad8(dim)], the rotated part into lat [heads, rows, row] f32,
+ * laid out like a cache row, whose first `rank` elements a product with the transposed key expansion fills. */
+int tilert_gqa_latent_queries_op(TgContext* ctx, const float* q, long long ldq, int rows, int heads, int dim, int rot,
+                                 const float* rope, int positions, int rope_dims, int interleaved, const int* pos, void* out,
+                                 float* lat, int rank, int f32, void* stream);
+/* Absorbed queries q [heads, tokens, row] f32 against the visible cache rows; token t is at *pos + t.  The key range is
+ * shared by n_splits CTAs; part gets [heads, tokens, n_splits, rankp] unnormalised sums of latents, then [.., 2] (largest
+ * score, sum of exponentials). */
+int tilert_gqa_latent_attn_op(TgContext* ctx, const float* q, const void* cache, int tokens, int heads, int rank, int rot,
+                              const int* pos, int window, int ring, float scale, int n_splits, float* part, int f32,
+                              void* stream);
+/* Parts -> out [heads, tokens, ldo]; sink [heads] or NULL: exp(sink) is one more term of the denominator. */
+int tilert_gqa_latent_merge_op(TgContext* ctx, const float* part, int tokens, int heads, int n_splits, int rank, int rot,
+                               const float* sink, void* out, long long ldo, int f32, void* stream);
+/* out[t, h * vdim + v] = o[h, t, v] * sigmoid(gate[t, h]) (per_head) or sigmoid(gate[t, h * vdim + v]); gate NULL: 1. */
+int tilert_gqa_gate_heads_op(TgContext* ctx, const float* o, int ldv, int rows, int heads, int vdim, const float* gate,
+                             long long ldg, int per_head, void* out, long long ldo, int f32, void* stream);
+/* The expanded form on bf16 tiles: kv [ring, heads * pad16(dim) | heads * pad16(vdim)] holds the keys and values of the
+ * cache rows in use, the rotated key part is read from the cache.  Sink and gate as above, out [rows, heads * vdim]. */
+int tilert_gqa_expanded_attn_op(TgContext* ctx, const void* q, const void* kv, const void* cache, int rows, int heads, int dim,
+                                int rot, int vdim, int rank, const int* pos, int window, int ring, float scale,
+                                const float* sink, const float* gate, long long ldg, int per_head, void* out, long long ldo,
+                                void* stream);
+/* One token: lat[h] = [w[h] q[h] | rotated part] with w [heads][rank][ldw] the transposed key expansion, and the cache
+ * row of *pos from the latent c and the key part kr. */
+int tilert_gqa_vec_absorb_op(TgContext* ctx, const float* q, int heads, int dim, int rank, int rot, const void* w, long long ldw,
+                             const float* rope, int positions, int rope_dims, int interleaved, const float* c, const float* kr,
+                             const float* c_gain, float eps, const int* pos, int ring, float* lat, void* cache, int f32,
+                             void* stream);
+/* One token: the merge of its parts, the value expansion w [heads][vdim][ldw] and the gate, out [heads * vdim]. */
+int tilert_gqa_vec_value_op(TgContext* ctx, const float* part, int heads, int vdim, int rank, int rot, int n_splits,
+                            const float* sink, const void* w, long long ldw, const float* gate, int per_head, float* out,
+                            void* stream);
 
 /* tilert_sample_op of tilert_b200.h (same kernel, same arguments). */
 int tilert_gqa_sample_op(TgContext* ctx, const float* logits, long long logits_stride, int tokens, int vocab,

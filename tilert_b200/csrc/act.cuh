@@ -48,4 +48,14 @@ __device__ __forceinline__ float clamped_gate(float gate, float up, float limit,
   return g / (1.f + expf(-alpha * g)) * (u + 1.f);
 }
 
+// An output gate: one value per head, or one per element of every head.
+struct HeadGate {
+  const float* z;        // [rows, ld]; null: no gate
+  long long ld;
+  int per_head;
+  __device__ __forceinline__ float operator()(int t, int h, int vdim, int v) const {
+    return z == nullptr ? 1.f : 1.f / (1.f + expf(-z[t * ld + (per_head ? h : h * vdim + v)]));
+  }
+};
+
 }  // namespace tb

@@ -25,9 +25,9 @@ constexpr int kMaxGroups = 1024;
 struct GemmRowsParams {
   int n;                 // output features
   int k;
-  int rows;              // token rows; grouped: an upper bound is not needed, the counts say how many
+  int rows;              // token rows; grouped with counts: an upper bound is not needed, the counts say how many
   int n_groups;          // 0: one weight for all rows
-  const int* counts;     // [n_groups] device
+  const int* counts;     // [n_groups] device; null: `rows` rows in every group
   float limit, alpha;    // GATED
   const float* bias;     // optional [n] (one weight only)
   void* out;
@@ -73,7 +73,7 @@ __device__ __forceinline__ void tile_prefix(const GemmRowsParams& p, int bn, int
     int r0 = 0, t0 = 0;
     for (int b = 0; b < p.n_groups; b += 32) {
       const int e = b + static_cast<int>(threadIdx.x);
-      const int c = e < p.n_groups ? p.counts[e] : 0;
+      const int c = e >= p.n_groups ? 0 : (p.counts != nullptr ? p.counts[e] : p.rows);
       int r = c, t = (c + bn - 1) / bn * ft;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {

@@ -1,4 +1,5 @@
-// C ABI of the grouped-query attention / mixture-of-experts path: argument checks and kernel launches.
+// C ABI of the decoders with bf16 weight rows (grouped-query and latent attention, dense and routed feed-forwards):
+// argument checks and kernel launches.
 // Declarations: include/tilert_gqa.h.
 #include "../../include/tilert_gqa.h"
 
@@ -10,6 +11,8 @@
 #include "host_util.h"
 
 #include "gemm_rows.cuh"
+#include "latent_attention.cuh"
+#include "latent_rows.cuh"
 #include "moe_rows.cuh"
 #include "norm_rows.cuh"
 #include "rowvec.cuh"
@@ -77,7 +80,8 @@ template <int BN, bool GATED>
 int launch_tc(TgContext* ctx, const GemmRowsParams& p, long long w_rows, void* stream) {
   CUtensorMap wmap, xmap;
   int rc = make_map(&wmap, p.w, w_rows, p.k, p.ldw, 128);
-  if (rc == TB_OK) rc = make_map(&xmap, p.x, p.rows, p.k, p.ldx, BN);
+  const long long x_rows = p.n_groups > 0 && p.counts == nullptr ? static_cast<long long>(p.n_groups) * p.rows : p.rows;
+  if (rc == TB_OK) rc = make_map(&xmap, p.x, x_rows, p.k, p.ldx, BN);
   if (rc != TB_OK) return rc;
   return go(gemm_tc_kernel<BN, GATED>, dim3(ctx->num_sms), dim3(kTcThreads), TcShape<BN, GATED>::kSmemBytes, stream, wmap, xmap, p);
 }
@@ -143,7 +147,7 @@ extern "C" int tilert_gqa_set_wait_budget(TgContext* ctx, long long cycles) {
 extern "C" int tilert_gqa_embed_norm_op(TgContext* ctx, const long long* tokens, const void* table, long long ld_table, int vocab,
                                         const float* gain, float eps, int rows, int dim, float* x, long long ldx, void* xh,
                                         long long ldh, int f32, void* stream) {
-  TB_REQUIRE(ctx != nullptr && tokens != nullptr && table != nullptr && gain != nullptr && x != nullptr);
+  TB_REQUIRE(ctx != nullptr && tokens != nullptr && table != nullptr && x != nullptr);
   TB_REQUIRE(rows >= 1 && dim >= 1 && vocab >= 1 && ld_table >= dim && ldx >= dim && (xh == nullptr || ldh >= dim));
   const EmbedNormParams p{tokens, reinterpret_cast<const __nv_bfloat16*>(table), ld_table, vocab, gain, eps, dim, x, ldx, xh, ldh,
                           ctx->status};
@@ -153,23 +157,27 @@ extern "C" int tilert_gqa_embed_norm_op(TgContext* ctx, const long long* tokens,
 
 extern "C" int tilert_gqa_residual_norm_op(TgContext* ctx, const float* y, long long ldy, const void* ye, long long lde,
                                            const int* slot_row, const float* slot_w, int top, const void* ysh, long long ldsh,
-                                           const float* gain, float eps, int rows, int dim, float* x, long long ldx, void* xh,
-                                           long long ldh, int f32, void* stream) {
-  TB_REQUIRE(ctx != nullptr && gain != nullptr && x != nullptr && xh != nullptr && rows >= 1 && dim >= 1 && ldx >= dim && ldh >= dim);
+                                           const float* gain, const float* bias, const float* add, const float* gain2,
+                                           const float* bias2, int centered, float eps, int rows, int dim, float* x, long long ldx,
+                                           void* xh, long long ldh, int f32, void* stream) {
+  TB_REQUIRE(ctx != nullptr && x != nullptr && rows >= 1 && dim >= 1 && ldx >= dim && (xh == nullptr || ldh >= dim));
+  TB_REQUIRE((gain != nullptr) == (y != nullptr || ye != nullptr) && (bias == nullptr || gain != nullptr));
+  TB_REQUIRE((gain2 == nullptr || xh != nullptr) && (bias2 == nullptr || gain2 != nullptr));
   TB_REQUIRE(y != nullptr ? ldy >= dim
-                          : (ye != nullptr && slot_row != nullptr && slot_w != nullptr && top >= 1 && stride_ok(lde, dim) && aligned16(ye) &&
-                             (ysh == nullptr || (stride_ok(ldsh, dim) && aligned16(ysh)))));
-  const ResidualNormParams p{y, ldy, ye, lde, slot_row, slot_w, top, ysh, ldsh, gain, eps, dim, x, ldx, xh, ldh};
+                          : (ye == nullptr || (slot_row != nullptr && slot_w != nullptr && top >= 1 && stride_ok(lde, dim) && aligned16(ye) &&
+                                               (ysh == nullptr || (stride_ok(ldsh, dim) && aligned16(ysh))))));
+  const ResidualNormParams p{y,    ldy, ye,    lde,   slot_row, slot_w, top, ysh, ldsh, gain, bias,
+                             add,  gain2, bias2, centered, eps, dim,    x,   ldx, xh,   ldh};
   const size_t smem = static_cast<size_t>(dim) * sizeof(float);
   if (f32) return go(residual_norm_kernel<float>, dim3(rows), dim3(kNormThreads), smem, stream, p);
   return go(residual_norm_kernel<__nv_bfloat16>, dim3(rows), dim3(kNormThreads), smem, stream, p);
 }
 
 extern "C" int tilert_gqa_gather_norm_op(TgContext* ctx, const float* x, long long ldx, const int* rows, int n, const float* gain,
-                                         float eps, int dim, void* out, long long ldo, int f32, void* stream) {
+                                         const float* bias, int centered, float eps, int dim, void* out, long long ldo, int f32, void* stream) {
   TB_REQUIRE(ctx != nullptr && x != nullptr && rows != nullptr && gain != nullptr && out != nullptr);
   TB_REQUIRE(n >= 1 && dim >= 1 && ldx >= dim && ldo >= dim);
-  const GatherNormParams p{x, ldx, rows, gain, eps, dim, out, ldo};
+  const GatherNormParams p{x, ldx, rows, gain, bias, centered, eps, dim, out, ldo};
   if (f32) return go(gather_norm_kernel<float>, dim3(n), dim3(kNormThreads), 0, stream, p);
   return go(gather_norm_kernel<__nv_bfloat16>, dim3(n), dim3(kNormThreads), 0, stream, p);
 }
@@ -179,7 +187,7 @@ extern "C" int tilert_gqa_gemm_op(TgContext* ctx, const void* x, long long ldx, 
                                   int gated, float limit, float alpha, int n_groups, const int* counts, const float* bias, void* out,
                                   long long ldo, int out_f32, int f32, void* stream) {
   TB_REQUIRE(ctx != nullptr && x != nullptr && w != nullptr && out != nullptr);
-  TB_REQUIRE(rows >= 1 && n >= 1 && k >= 1 && n_groups >= 0 && n_groups <= kMaxGroups && (n_groups == 0 || counts != nullptr));
+  TB_REQUIRE(rows >= 1 && n >= 1 && k >= 1 && n_groups >= 0 && n_groups <= kMaxGroups);
   TB_REQUIRE(stride_ok(ldx, k) && stride_ok(ldw, k) && ldo >= n && aligned16(x) && aligned16(w));
   TB_REQUIRE(bias == nullptr || (n_groups == 0 && !gated));
   const int per = gated ? 2 : 1;
@@ -211,7 +219,7 @@ extern "C" int tilert_gqa_gemm_op(TgContext* ctx, const void* x, long long ldx, 
   // Token tile.  One weight: waves of tiles over the SMs times the relative cost of a tile (a narrow tile moves more
   // bytes per product through the L2).  Groups: the widest tile that an average group nearly fills.
   auto cost = [&](int bn, double tile) {
-    if (n_groups > 0) return bn == 64 || rows / n_groups >= bn * 3 / 4 ? 1.0 / bn : 1.0;
+    if (n_groups > 0) return bn == 64 || (counts != nullptr ? rows / n_groups : rows) >= bn * 3 / 4 ? 1.0 / bn : 1.0;
     return std::ceil(static_cast<double>(ft) * ((rows + bn - 1) / bn) / ctx->num_sms) * tile;
   };
   if (gated) return cost(128, 1.0) <= cost(64, 0.6) ? launch_tc<128, true>(ctx, p, w_rows, stream) : launch_tc<64, true>(ctx, p, w_rows, stream);
@@ -254,6 +262,16 @@ int launch_prefill_attn(const AttnPrefillParams& p, dim3 grid, void* stream) {
   return go(attn_prefill_kernel<DV16>, grid, dim3(kFaThreads), attn_prefill_smem(p.s.dimp, p.s.vdimp), stream, p);
 }
 
+bool prefill_attn_fits(int dimp, int vdimp) { return vdimp <= 256 && attn_prefill_smem(dimp, vdimp) <= kMaxSmem; }
+
+int run_prefill_attn(const AttnPrefillParams& p, void* stream) {
+  const int group = p.s.heads / p.s.kv_heads, hpb = group < kFaMaxHeads ? group : kFaMaxHeads, tpb = kFaRows / hpb;
+  const dim3 grid((p.rows + tpb - 1) / tpb, p.s.kv_heads * ((group + hpb - 1) / hpb));
+  if (p.s.vdimp <= 64) return launch_prefill_attn<4>(p, grid, stream);
+  if (p.s.vdimp <= 128) return launch_prefill_attn<8>(p, grid, stream);
+  return launch_prefill_attn<16>(p, grid, stream);
+}
+
 }  // namespace
 
 extern "C" int tilert_gqa_head_blocks(int heads, int kv_heads) { return head_blocks(heads, kv_heads); }
@@ -266,7 +284,7 @@ extern "C" int tilert_gqa_attn_rows_op(TgContext* ctx, const void* q, const void
   if (rc != TB_OK) return rc;
   TB_REQUIRE(ctx != nullptr && q != nullptr && k_cache != nullptr && v_cache != nullptr && pos != nullptr && out != nullptr);
   TB_REQUIRE(rows >= 1 && ldo >= static_cast<long long>(heads) * vdim && window + rows - 1 <= ring);
-  if (!f32 && s.vdimp <= 256 && attn_prefill_smem(s.dimp, s.vdimp) <= kMaxSmem) {
+  if (!f32 && prefill_attn_fits(s.dimp, s.vdimp)) {
     AttnPrefillParams p{};
     p.s = s;
     p.pos = pos;
@@ -274,21 +292,25 @@ extern "C" int tilert_gqa_attn_rows_op(TgContext* ctx, const void* q, const void
     p.q = reinterpret_cast<const __nv_bfloat16*>(q);
     p.k_cache = reinterpret_cast<const __nv_bfloat16*>(k_cache);
     p.v_cache = reinterpret_cast<const __nv_bfloat16*>(v_cache);
+    p.k_ld = p.dim1 = s.dimp;
+    p.v_ld = s.vdimp;
+    p.k_head = static_cast<long long>(ring) * s.dimp;
+    p.v_head = static_cast<long long>(ring) * s.vdimp;
     p.scale = scale;
     p.out = reinterpret_cast<__nv_bfloat16*>(out);
     p.ldo = ldo;
-    const int group = heads / kv_heads, hpb = group < kFaMaxHeads ? group : kFaMaxHeads, tpb = kFaRows / hpb;
-    const dim3 grid((rows + tpb - 1) / tpb, kv_heads * ((group + hpb - 1) / hpb));
-    if (s.vdimp <= 64) return launch_prefill_attn<4>(p, grid, stream);
-    if (s.vdimp <= 128) return launch_prefill_attn<8>(p, grid, stream);
-    return launch_prefill_attn<16>(p, grid, stream);
+    return run_prefill_attn(p, stream);
   }
   AttnRowsParams a{};
   a.s = s;
   a.pos = pos;
   a.q = q;
+  a.q_head = s.dimp;
+  a.q_token = static_cast<long long>(heads) * s.dimp;
   a.k_cache = const_cast<void*>(k_cache);
   a.v_cache = const_cast<void*>(v_cache);
+  a.v_ld = s.vdimp;
+  a.rows = rows;
   a.scale = scale;
   a.n_splits = 1;
   a.out = out;
@@ -323,15 +345,42 @@ extern "C" int tilert_gqa_gather_rows_op(TgContext* ctx, const void* x, long lon
 }
 
 // ------------------------------------------------------------------------------- one-token step
-extern "C" int tilert_gqa_vec_dense_op(TgContext* ctx, const float* x, const float* y, const float* gain, const float* gain2, float eps,
+namespace {
+
+int check_stage(const RvStage& s) {
+  TB_REQUIRE(s.x != nullptr && s.k >= 1 && (s.y == nullptr) == (s.gain == nullptr) && (s.bias == nullptr || s.gain != nullptr));
+  TB_REQUIRE((s.bias2 == nullptr || s.gain2 != nullptr) && (s.x_out == nullptr || (s.x_out != s.x && s.x_out != s.y)));
+  TB_REQUIRE(aligned16(s.x) && aligned16(s.y) && aligned16(s.gain) && aligned16(s.bias) && aligned16(s.add) && aligned16(s.gain2) &&
+             aligned16(s.bias2) && aligned16(s.x_out));
+  return TB_OK;
+}
+
+}  // namespace
+
+extern "C" int tilert_gqa_vec_dense_op(TgContext* ctx, const float* x, const float* y, const float* gain, const float* norm_bias,
+                                       const float* add, const float* gain2, const float* norm_bias2, int centered, float eps,
                                        float* x_out, const void* w, long long ldw, const float* bias, int n, int k, float* out,
                                        void* stream) {
-  TB_REQUIRE(ctx != nullptr && x != nullptr && w != nullptr && out != nullptr && n >= 1 && k >= 1);
-  TB_REQUIRE((y == nullptr) == (gain == nullptr) && (x_out == nullptr || (x_out != x && x_out != y)));
-  TB_REQUIRE(stride_ok(ldw, k) && aligned16(w) && aligned16(x));
-  const RvDenseParams p{{x, y, gain, gain2, x_out, eps, k}, reinterpret_cast<const __nv_bfloat16*>(w), ldw, bias, n, out};
+  const RvStage in{x, y, gain, norm_bias, add, gain2, norm_bias2, x_out, eps, centered, k};
+  const int rc = check_stage(in);
+  if (rc != TB_OK) return rc;
+  TB_REQUIRE(ctx != nullptr && w != nullptr && out != nullptr && n >= 1 && stride_ok(ldw, k) && aligned16(w));
+  const RvDenseParams p{in, reinterpret_cast<const __nv_bfloat16*>(w), ldw, bias, n, out};
   const int grid = n < ctx->num_sms ? n : ctx->num_sms;
   return go(rv_dense_kernel, dim3(grid), dim3(kRvThreads), kRvPartBytes + rv_vec_bytes(pad_to(k, 8)), stream, p);
+}
+
+extern "C" int tilert_gqa_vec_gated_op(TgContext* ctx, const float* x, const float* y, const float* gain, const float* norm_bias,
+                                       const float* add, const float* gain2, const float* norm_bias2, int centered, float eps,
+                                       float* x_out, const void* w, long long ldw, int n, int k, float limit, float alpha, float* out,
+                                       void* stream) {
+  const RvStage in{x, y, gain, norm_bias, add, gain2, norm_bias2, x_out, eps, centered, k};
+  const int rc = check_stage(in);
+  if (rc != TB_OK) return rc;
+  TB_REQUIRE(ctx != nullptr && w != nullptr && out != nullptr && n >= 1 && stride_ok(ldw, k) && aligned16(w));
+  const RvGatedParams p{in, reinterpret_cast<const __nv_bfloat16*>(w), ldw, n, limit, alpha, out};
+  const int grid = n < ctx->num_sms ? n : ctx->num_sms;
+  return go(rv_gated_kernel, dim3(grid), dim3(kRvThreads), kRvPartBytes + rv_vec_bytes(pad_to(k, 8)), stream, p);
 }
 
 extern "C" int tilert_gqa_vec_attn_op(TgContext* ctx, const float* qkv, const float* q_gain, const float* k_gain, float eps, int v_mode,
@@ -350,6 +399,8 @@ extern "C" int tilert_gqa_vec_attn_op(TgContext* ctx, const float* qkv, const fl
   a.pos = pos;
   a.k_cache = k_cache;
   a.v_cache = v_cache;
+  a.v_ld = a.s.vdimp;
+  a.rows = 1;
   a.scale = scale;
   a.n_splits = n_splits;
   a.part = part;
@@ -385,6 +436,257 @@ extern "C" int tilert_gqa_vec_down_op(TgContext* ctx, const float* hidden, const
   const int kp = pad_to(ff_sh, 8) + top * pad_to(ff, 8);
   const int grid = dim < ctx->num_sms ? dim : ctx->num_sms;
   return go(rv_down_kernel, dim3(grid), dim3(kRvThreads), kRvPartBytes + rv_vec_bytes(kp) + sizeof(RvPiece) * (kp / 8), stream, p);
+}
+
+// ------------------------------------------------------------------------------- attention over a latent cache
+namespace {
+
+LatentRow latent_row(int rank, int rot) {
+  const int rankp = pad_to(rank, 16);
+  return {rank, rankp, rot, pad_to(rankp + rot, 32)};
+}
+int check_latent(const LatentRow& r, int heads, int ring) {
+  TB_REQUIRE(r.rank >= 1 && r.rank <= 2048 && r.rot >= 1 && r.row <= 4096 && heads >= 1 && heads <= kMaxGroups && ring >= 1);
+  return TB_OK;
+}
+int check_rotation(const Rotation& r, int rot) {
+  TB_REQUIRE(r.table != nullptr && r.positions >= 1 && r.dims >= 0 && r.dims % 2 == 0 && r.dims <= rot);
+  return TB_OK;
+}
+
+// Tiles of 16 query rows per CTA of the tensor-core kernel; 0: its tiles do not fit, the row kernel runs
+int latent_tiles(int n_rows, const LatentRow& r) {
+  if (r.rankp > 1024) return 0;
+  if (n_rows > 16 && latent_attn_smem(2, r.row) <= kMaxSmem) return 2;
+  return latent_attn_smem(1, r.row) <= kMaxSmem ? 1 : 0;
+}
+
+template <int MT>
+int launch_latent(const LatentAttnParams& p, void* stream) {
+  const dim3 grid(p.n_splits, (p.n_rows + 16 * MT - 1) / (16 * MT));
+  const size_t smem = latent_attn_smem(MT, p.r.row);
+  if (p.r.rankp <= 128) return go(latent_attn_kernel<MT, 1>, grid, dim3(kLaThreads), smem, stream, p);
+  if (p.r.rankp <= 256) return go(latent_attn_kernel<MT, 2>, grid, dim3(kLaThreads), smem, stream, p);
+  if (p.r.rankp <= 512) return go(latent_attn_kernel<MT, 4>, grid, dim3(kLaThreads), smem, stream, p);
+  return go(latent_attn_kernel<MT, 8>, grid, dim3(kLaThreads), smem, stream, p);
+}
+
+}  // namespace
+
+extern "C" int tilert_gqa_latent_row_len(int rank, int rot) { return latent_row(rank, rot).row; }
+
+extern "C" int tilert_gqa_latent_blocks(int heads, int tokens, int rank, int rot, int f32) {
+  const int mt = f32 ? 0 : latent_tiles(heads * tokens, latent_row(rank, rot));
+  return mt > 0 ? (heads * tokens + 16 * mt - 1) / (16 * mt) : head_blocks(heads, 1) * tokens;
+}
+
+extern "C" int tilert_gqa_expanded_fits(int dim, int rot, int vdim) {
+  return prefill_attn_fits(pad_to(dim, 16) + pad_to(rot, 16), pad_to(vdim, 16)) ? 1 : 0;
+}
+
+extern "C" int tilert_gqa_latent_tokens_op(TgContext* ctx, const float* z, long long ldz, int q_rank, int off_c, int off_r,
+                                           const float* q_gain, const float* c_gain, float eps, int rows, int rank, int rot,
+                                           const float* rope, int positions, int rope_dims, int interleaved, const int* pos, int ring,
+                                           void* cq, long long ldq, void* cache, int f32, void* stream) {
+  LatentTokensParams p{};
+  p.r = latent_row(rank, rot);
+  p.rope = {rope, positions, rope_dims, interleaved};
+  int rc = check_latent(p.r, 1, ring);
+  if (rc == TB_OK) rc = check_rotation(p.rope, rot);
+  if (rc != TB_OK) return rc;
+  TB_REQUIRE(ctx != nullptr && z != nullptr && q_gain != nullptr && c_gain != nullptr && pos != nullptr && cq != nullptr && cache != nullptr);
+  TB_REQUIRE(rows >= 1 && rows <= ring && q_rank >= 1 && ldq >= q_rank && off_c >= 0 && off_r >= 0 && ldz >= off_c + rank && ldz >= off_r + rot);
+  p.z = z;
+  p.ldz = ldz;
+  p.q_rank = q_rank;
+  p.off_c = off_c;
+  p.off_r = off_r;
+  p.q_gain = q_gain;
+  p.c_gain = c_gain;
+  p.eps = eps;
+  p.pos = pos;
+  p.ring = ring;
+  p.cq = cq;
+  p.ldq = ldq;
+  p.cache = cache;
+  if (f32) return go(latent_tokens_kernel<float>, dim3(rows), dim3(256), 0, stream, p);
+  return go(latent_tokens_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, stream, p);
+}
+
+extern "C" int tilert_gqa_latent_queries_op(TgContext* ctx, const float* q, long long ldq, int rows, int heads, int dim, int rot,
+                                            const float* rope, int positions, int rope_dims, int interleaved, const int* pos, void* out,
+                                            float* lat, int rank, int f32, void* stream) {
+  LatentQueriesParams p{};
+  p.rope = {rope, positions, rope_dims, interleaved};
+  const int rc = check_rotation(p.rope, rot);
+  if (rc != TB_OK) return rc;
+  TB_REQUIRE(ctx != nullptr && q != nullptr && pos != nullptr && out != nullptr && rows >= 1 && heads >= 1 && dim >= 1 && rot >= 1);
+  TB_REQUIRE(lat == nullptr || rank >= 1);
+  p.q = q;
+  p.ldq = ldq;
+  p.heads = heads;
+  p.dim = dim;
+  p.dimp8 = pad_to(dim, 8);
+  p.rot = rot;
+  p.ldh = p.dimp8 + pad_to(rot, 8);
+  TB_REQUIRE(ldq >= static_cast<long long>(heads) * p.ldh);
+  p.pos = pos;
+  p.rows = rows;
+  p.out = out;
+  p.wide = pad_to(dim, 16) + pad_to(rot, 16);
+  p.lat = lat;
+  if (lat != nullptr) {
+    const LatentRow r = latent_row(rank, rot);
+    p.off_rot = r.rankp;
+    p.row = r.row;
+  } else {
+    p.off_rot = pad_to(dim, 16);
+  }
+  if (f32) return go(latent_queries_kernel<float>, dim3(rows), dim3(256), 0, stream, p);
+  return go(latent_queries_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, stream, p);
+}
+
+extern "C" int tilert_gqa_latent_attn_op(TgContext* ctx, const float* q, const void* cache, int tokens, int heads, int rank, int rot,
+                                         const int* pos, int window, int ring, float scale, int n_splits, float* part, int f32,
+                                         void* stream) {
+  const LatentRow r = latent_row(rank, rot);
+  const int rc = check_latent(r, heads, ring);
+  if (rc != TB_OK) return rc;
+  TB_REQUIRE(ctx != nullptr && q != nullptr && cache != nullptr && pos != nullptr && part != nullptr && aligned16(q) && aligned16(cache) && aligned16(part));
+  TB_REQUIRE(tokens >= 1 && tokens <= 32768 && window >= 0 && window + tokens - 1 <= ring && n_splits >= 1 && n_splits <= 1024);
+  const int mt = f32 ? 0 : latent_tiles(heads * tokens, r);
+  if (mt > 0) {
+    LatentAttnParams p{};
+    p.r = r;
+    p.n_rows = heads * tokens;
+    p.tokens = tokens;
+    p.ring = ring;
+    p.window = window;
+    p.pos = pos;
+    p.q = q;
+    p.cache = reinterpret_cast<const __nv_bfloat16*>(cache);
+    p.scale = scale;
+    p.n_splits = n_splits;
+    p.part = part;
+    return mt == 2 ? launch_latent<2>(p, stream) : launch_latent<1>(p, stream);
+  }
+  AttnRowsParams a{};
+  a.s = {heads, 1, r.row, r.rank, r.row, r.rankp, ring, window};
+  a.pos = pos;
+  a.q = q;
+  a.q_head = static_cast<long long>(tokens) * r.row;
+  a.q_token = r.row;
+  a.k_cache = a.v_cache = const_cast<void*>(cache);
+  a.v_ld = r.row;
+  a.rows = tokens;
+  a.scale = scale;
+  a.n_splits = n_splits;
+  a.part = part;
+  a.parts_only = 1;
+  const dim3 grid(n_splits, head_blocks(heads, 1), tokens);
+  const size_t smem = attn_rows_smem(r.row, r.rankp);
+  if (f32) return go(attn_rows_kernel<float, false, float>, grid, dim3(kAttnThreads), smem, stream, a);
+  return go(attn_rows_kernel<__nv_bfloat16, false, float>, grid, dim3(kAttnThreads), smem, stream, a);
+}
+
+extern "C" int tilert_gqa_latent_merge_op(TgContext* ctx, const float* part, int tokens, int heads, int n_splits, int rank, int rot,
+                                          const float* sink, void* out, long long ldo, int f32, void* stream) {
+  const LatentRow r = latent_row(rank, rot);
+  TB_REQUIRE(ctx != nullptr && part != nullptr && out != nullptr && tokens >= 1 && heads >= 1 && n_splits >= 1 && n_splits <= 1024 && ldo >= rank);
+  const LatentMergeParams p{part, heads * tokens, tokens, n_splits, rank, r.rankp, sink, out, ldo};
+  const size_t smem = sizeof(float) * n_splits;
+  if (f32) return go(latent_merge_kernel<float>, dim3(heads * tokens), dim3(128), smem, stream, p);
+  return go(latent_merge_kernel<__nv_bfloat16>, dim3(heads * tokens), dim3(128), smem, stream, p);
+}
+
+extern "C" int tilert_gqa_gate_heads_op(TgContext* ctx, const float* o, int ldv, int rows, int heads, int vdim, const float* gate,
+                                        long long ldg, int per_head, void* out, long long ldo, int f32, void* stream) {
+  TB_REQUIRE(ctx != nullptr && o != nullptr && out != nullptr && rows >= 1 && heads >= 1 && vdim >= 1 && ldv >= vdim);
+  TB_REQUIRE(ldo >= static_cast<long long>(heads) * vdim && (gate == nullptr || ldg >= (per_head ? heads : heads * vdim)));
+  const GateHeadsParams p{o, ldv, heads, vdim, rows, {gate, ldg, per_head}, out, ldo};
+  if (f32) return go(gate_heads_kernel<float>, dim3(rows), dim3(256), 0, stream, p);
+  return go(gate_heads_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, stream, p);
+}
+
+extern "C" int tilert_gqa_expanded_attn_op(TgContext* ctx, const void* q, const void* kv, const void* cache, int rows, int heads, int dim,
+                                           int rot, int vdim, int rank, const int* pos, int window, int ring, float scale,
+                                           const float* sink, const float* gate, long long ldg, int per_head, void* out, long long ldo,
+                                           void* stream) {
+  const LatentRow r = latent_row(rank, rot);
+  const int rc = check_latent(r, heads, ring);
+  if (rc != TB_OK) return rc;
+  const int dimp = pad_to(dim, 16), rotp = pad_to(rot, 16), vdimp = pad_to(vdim, 16);
+  TB_REQUIRE(ctx != nullptr && q != nullptr && kv != nullptr && cache != nullptr && pos != nullptr && out != nullptr && rows >= 1);
+  TB_REQUIRE(aligned16(q) && aligned16(kv) && aligned16(cache) && dim >= 1 && vdim >= 1 && window >= 0 && window + rows - 1 <= ring);
+  TB_REQUIRE(prefill_attn_fits(dimp + rotp, vdimp) && ldo >= static_cast<long long>(heads) * vdim && (vdim % 2 == 1 || ldo % 2 == 0));
+  TB_REQUIRE(gate == nullptr || ldg >= (per_head ? heads : heads * vdim));
+  AttnPrefillParams p{};
+  p.s = {heads, heads, dim + rot, vdim, dimp + rotp, vdimp, ring, window};
+  p.pos = pos;
+  p.rows = rows;
+  p.q = reinterpret_cast<const __nv_bfloat16*>(q);
+  p.k_cache = reinterpret_cast<const __nv_bfloat16*>(kv);
+  p.v_cache = p.k_cache + static_cast<long long>(heads) * dimp;
+  p.k2 = reinterpret_cast<const __nv_bfloat16*>(cache) + r.rankp;
+  p.k_head = p.dim1 = dimp;
+  p.v_head = vdimp;
+  p.k_ld = p.v_ld = static_cast<long long>(heads) * (dimp + vdimp);
+  p.k2_ld = r.row;
+  p.scale = scale;
+  p.sink = sink;
+  p.gate = {gate, ldg, gate != nullptr ? per_head : 0};
+  p.out = reinterpret_cast<__nv_bfloat16*>(out);
+  p.ldo = ldo;
+  return run_prefill_attn(p, stream);
+}
+
+extern "C" int tilert_gqa_vec_absorb_op(TgContext* ctx, const float* q, int heads, int dim, int rank, int rot, const void* w, long long ldw,
+                                        const float* rope, int positions, int rope_dims, int interleaved, const float* c, const float* kr,
+                                        const float* c_gain, float eps, const int* pos, int ring, float* lat, void* cache, int f32,
+                                        void* stream) {
+  RvAbsorbParams p{};
+  p.r = latent_row(rank, rot);
+  p.rope = {rope, positions, rope_dims, interleaved};
+  int rc = check_latent(p.r, heads, ring);
+  if (rc == TB_OK) rc = check_rotation(p.rope, rot);
+  if (rc != TB_OK) return rc;
+  TB_REQUIRE(ctx != nullptr && q != nullptr && w != nullptr && c != nullptr && kr != nullptr && c_gain != nullptr && pos != nullptr && lat != nullptr && cache != nullptr);
+  TB_REQUIRE(dim >= 1 && stride_ok(ldw, dim) && aligned16(w) && aligned16(q) && aligned16(lat) && aligned16(cache));
+  p.q = q;
+  p.heads = heads;
+  p.dim = dim;
+  p.dimp8 = pad_to(dim, 8);
+  p.ldh = p.dimp8 + pad_to(rot, 8);
+  p.w = reinterpret_cast<const __nv_bfloat16*>(w);
+  p.ldw = ldw;
+  p.c = c;
+  p.kr = kr;
+  p.c_gain = c_gain;
+  p.eps = eps;
+  p.pos = pos;
+  p.ring = ring;
+  p.lat = lat;
+  p.cache = cache;
+  const long long groups = static_cast<long long>(heads) * ((rank + 3) / 4);
+  const int grid = groups < ctx->num_sms ? static_cast<int>(groups) : ctx->num_sms;
+  const size_t smem = kRvPartBytes + sizeof(float) * rv_heads_span(heads, rank, grid) * rv_vec_stride(p.dimp8);
+  if (f32) return go(rv_absorb_kernel<float>, dim3(grid), dim3(kRvThreads), smem, stream, p);
+  return go(rv_absorb_kernel<__nv_bfloat16>, dim3(grid), dim3(kRvThreads), smem, stream, p);
+}
+
+extern "C" int tilert_gqa_vec_value_op(TgContext* ctx, const float* part, int heads, int vdim, int rank, int rot, int n_splits,
+                                       const float* sink, const void* w, long long ldw, const float* gate, int per_head, float* out,
+                                       void* stream) {
+  const LatentRow r = latent_row(rank, rot);
+  const int rc = check_latent(r, heads, 1);
+  if (rc != TB_OK) return rc;
+  TB_REQUIRE(ctx != nullptr && part != nullptr && w != nullptr && out != nullptr && vdim >= 1 && n_splits >= 1 && n_splits <= 1024);
+  TB_REQUIRE(stride_ok(ldw, rank) && aligned16(w) && aligned16(part));
+  const RvValueParams p{r, part, heads, vdim, n_splits, sink, reinterpret_cast<const __nv_bfloat16*>(w), ldw, {gate, 0, per_head}, out};
+  const long long groups = static_cast<long long>(heads) * ((vdim + 3) / 4);
+  const int grid = groups < ctx->num_sms ? static_cast<int>(groups) : ctx->num_sms;
+  const size_t smem = kRvPartBytes + sizeof(float) * rv_heads_span(heads, vdim, grid) * (rv_vec_stride(pad_to(rank, 8)) + n_splits);
+  return go(rv_value_kernel, dim3(grid), dim3(kRvThreads), smem, stream, p);
 }
 
 // ------------------------------------------------------------------------------- sampling

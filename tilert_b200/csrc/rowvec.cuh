@@ -1,6 +1,7 @@
 // Single-token products: one activation vector (f32) against bf16 weights, bound by the weight stream from HBM.
 //
 //   dense     out[n] = W[n, :] . x (+ bias)
+//   gated     hidden[n] = clamped_gate(W_gate[n, :] . x, W_up[n, :] . x)
 //   gate/up   routing, then hidden = clamped_gate(W_gate x, W_up x) of the shared and the selected experts
 //   down      out[d] = sum over slots of w_slot W_down[slot][d, :] . hidden[slot]
 //
@@ -10,9 +11,10 @@
 // flight.  Four row sums are reduced across a warp together (transposing: six shuffles instead of twenty) and the
 // per-warp sums of a team meet in shared memory at the end.
 //
-// The vector is staged once per CTA.  Staging can apply what lies between two sublayers -- x + rms(y) gain, written
-// back by CTA 0, and a further norm on top -- so that the norms and the residual of a decode step need no launches of
-// their own.  Weights that do not depend on the predecessor are requested before the wait for it.
+// The vector is staged once per CTA.  Staging can apply what lies between two sublayers -- x + norm(y) (+ a constant
+// vector), written back by CTA 0, and a further norm on top -- so that the norms and the residual of a decode step need
+// no launches of their own.  A norm is the RMS norm, or with `centered` the layer norm.  Weights that do not depend on
+// the predecessor are requested before the wait for it.
 #pragma once
 
 #include "act.cuh"
@@ -27,12 +29,16 @@ constexpr int kRvAhead = 2;        // steps requested beyond the current one
 constexpr int kRvBatchRows = 512;  // weight rows between two reductions over the warps
 
 struct RvStage {
-  const float* x;      // [pad8(k)], zero beyond k, as are y, gain and gain2
-  const float* y;      // optional sublayer output: the vector is x + rms(y) * gain
-  const float* gain;
+  const float* x;      // [pad8(k)], zero beyond k, as are y and all constants
+  const float* y;      // optional sublayer output: the vector is x + norm(y)
+  const float* gain;   // with y
+  const float* bias;   // optional, with y
+  const float* add;    // optional constant added to the vector
   const float* gain2;  // optional norm of the result
-  float* x_out;        // optional: CTA 0 stores x + rms(y) * gain (before gain2); must not alias x or y
+  const float* bias2;  // optional, with gain2
+  float* x_out;        // optional: CTA 0 stores the vector (before gain2); must not alias x or y
   float eps;
+  int centered;        // both norms
   int k;
 };
 
@@ -52,60 +58,98 @@ struct RvVec {
 };
 
 __device__ __forceinline__ float dot4(const float4& a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
+__device__ __forceinline__ float sum4(const float4& a) { return (a.x + a.y) + (a.z + a.w); }
+// (v - mean) * rinv * gain + bias
+__device__ __forceinline__ float4 norm4(const float4& v, float mean, float rinv, const float* gain, const float* bias, int g) {
+  const float4 c = reinterpret_cast<const float4*>(gain)[g];
+  const float4 b = bias != nullptr ? reinterpret_cast<const float4*>(bias)[g] : make_float4(0.f, 0.f, 0.f, 0.f);
+  return make_float4((v.x - mean) * rinv * c.x + b.x, (v.y - mean) * rinv * c.y + b.y, (v.z - mean) * rinv * c.z + b.z,
+                     (v.w - mean) * rinv * c.w + b.w);
+}
+
+// Statistics of the staged vector, every thread reading the groups it wrote itself; `first` is the thread's sum of
+// values (centered) or of squares.
+__device__ __forceinline__ void rv_stat(const RvVec& v, int k, float eps, int centered, float first, float* red, float& mean, float& rinv) {
+  float ss = first;
+  mean = 0.f;
+  if (centered) {
+    mean = cta_sum(first, red) / static_cast<float>(k);
+    ss = 0.f;
+    for (int g = threadIdx.x; g < pad_to(k, 8) / 4; g += kRvThreads) {
+      const float4 a = v.get4(g);
+      const float4 d = make_float4(a.x - mean, a.y - mean, a.z - mean, a.w - mean);
+      if (4 * g + 4 <= k) {
+        ss += dot4(d);
+      } else {  // the padding is no value
+        if (4 * g < k) ss += d.x * d.x;
+        if (4 * g + 1 < k) ss += d.y * d.y;
+        if (4 * g + 2 < k) ss += d.z * d.z;
+      }
+    }
+  }
+  rinv = 1.f / sqrtf(cta_sum(ss, red) / static_cast<float>(k) + eps);
+}
+
+// Constants of the staging, requested before the wait for the predecessor.
+__device__ __forceinline__ void rv_prefetch(const RvStage& s) {
+  const float* c[5] = {s.gain, s.bias, s.add, s.gain2, s.bias2};
+  for (int i = threadIdx.x * 32; i < s.k; i += kRvThreads * 32)
+#pragma unroll
+    for (int j = 0; j < 5; ++j)
+      if (c[j] != nullptr) asm volatile("prefetch.global.L1 [%0];" ::"l"(c[j] + i));
+}
 
 __device__ __forceinline__ void rv_stage(const RvStage& s, const RvVec& v, float* red) {
   constexpr int kReg = 4;  // groups of four per thread held in registers: k up to 8192 costs one round trip
   const int ng = pad_to(s.k, 8) / 4;
   const float4* x4 = reinterpret_cast<const float4*>(s.x);
   const float4* y4 = reinterpret_cast<const float4*>(s.y);
-  const float4* g4 = reinterpret_cast<const float4*>(s.gain);
-  const float4* h4 = reinterpret_cast<const float4*>(s.gain2);
-  float ss = 0.f;
+  float sum = 0.f, mean, rinv;
+  auto finish = [&](int g, float4 o) {  // the vector's group g is known: into shared memory, and out
+    if (s.add != nullptr) {
+      const float4 c = reinterpret_cast<const float4*>(s.add)[g];
+      o = make_float4(o.x + c.x, o.y + c.y, o.z + c.z, o.w + c.w);
+    }
+    v.put4(g, o);
+    sum += s.centered ? sum4(o) : dot4(o);
+    if (s.x_out != nullptr && blockIdx.x == 0) reinterpret_cast<float4*>(s.x_out)[g] = o;
+  };
   if (s.y != nullptr) {
-    float4 xr[kReg], yr[kReg], gr[kReg];
+    float4 xr[kReg], yr[kReg];
 #pragma unroll
     for (int i = 0; i < kReg; ++i) {
       const int g = threadIdx.x + i * kRvThreads;
       if (g < ng) {
         yr[i] = y4[g];
         xr[i] = x4[g];
-        gr[i] = g4[g];
       }
     }
-#pragma unroll
-    for (int i = 0; i < kReg; ++i)
-      if (threadIdx.x + i * kRvThreads < ng) ss += dot4(yr[i]);
-    for (int g = threadIdx.x + kReg * kRvThreads; g < ng; g += kRvThreads) ss += dot4(y4[g]);
-    const float rinv = 1.f / sqrtf(cta_sum(ss, red) / static_cast<float>(s.k) + s.eps);
-    ss = 0.f;
-    auto emit = [&](int g, const float4& a, const float4& b, const float4& c) {
-      const float4 o = make_float4(a.x + b.x * rinv * c.x, a.y + b.y * rinv * c.y, a.z + b.z * rinv * c.z, a.w + b.w * rinv * c.w);
-      v.put4(g, o);
-      ss += dot4(o);
-      if (s.x_out != nullptr && blockIdx.x == 0) reinterpret_cast<float4*>(s.x_out)[g] = o;
+    auto hold = [&](int g, const float4& a) {
+      v.put4(g, a);
+      sum += s.centered ? sum4(a) : dot4(a);
     };
 #pragma unroll
-    for (int i = 0; i < kReg; ++i) {
-      const int g = threadIdx.x + i * kRvThreads;
-      if (g < ng) emit(g, xr[i], yr[i], gr[i]);
-    }
-    for (int g = threadIdx.x + kReg * kRvThreads; g < ng; g += kRvThreads) emit(g, x4[g], y4[g], g4[g]);
+    for (int i = 0; i < kReg; ++i)
+      if (threadIdx.x + i * kRvThreads < ng) hold(threadIdx.x + i * kRvThreads, yr[i]);
+    for (int g = threadIdx.x + kReg * kRvThreads; g < ng; g += kRvThreads) hold(g, y4[g]);
+    rv_stat(v, s.k, s.eps, s.centered, sum, red, mean, rinv);
+    sum = 0.f;
+    auto emit = [&](int g, const float4& a) {
+      const float4 n = norm4(v.get4(g), mean, rinv, s.gain, s.bias, g);
+      finish(g, make_float4(a.x + n.x, a.y + n.y, a.z + n.z, a.w + n.w));
+    };
+#pragma unroll
+    for (int i = 0; i < kReg; ++i)
+      if (threadIdx.x + i * kRvThreads < ng) emit(threadIdx.x + i * kRvThreads, xr[i]);
+    for (int g = threadIdx.x + kReg * kRvThreads; g < ng; g += kRvThreads) emit(g, x4[g]);
   } else {
 #pragma unroll 4
-    for (int g = threadIdx.x; g < ng; g += kRvThreads) {
-      const float4 o = x4[g];
-      v.put4(g, o);
-      ss += dot4(o);
-    }
+    for (int g = threadIdx.x; g < ng; g += kRvThreads) finish(g, x4[g]);
   }
   if (s.gain2 != nullptr) {
-    const float rinv = 1.f / sqrtf(cta_sum(ss, red) / static_cast<float>(s.k) + s.eps);
-    for (int g = threadIdx.x; g < ng; g += kRvThreads) {  // every thread rescales what it wrote
-      float4 o = v.get4(g);
-      const float4 c = h4[g];
-      o = make_float4(o.x * rinv * c.x, o.y * rinv * c.y, o.z * rinv * c.z, o.w * rinv * c.w);
-      v.put4(g, o);
-    }
+    rv_stat(v, s.k, s.eps, s.centered, sum, red, mean, rinv);
+    for (int g = threadIdx.x; g < ng; g += kRvThreads)  // every thread rescales what it wrote
+      v.put4(g, norm4(v.get4(g), mean, rinv, s.gain2, s.bias2, g));
   }
   __syncthreads();
 }
@@ -155,9 +199,10 @@ __device__ __forceinline__ void rv_load(const Src& src, const RvTeam& t, const R
 }
 
 // Sums of `rows` weight rows (Src::load(row, piece)) against the staged vector into part[row][warp of the team].
-// `ahead` holds the first 1 + kRvAhead steps' weights when `loaded` is set.
-template <class Src>
-__device__ __forceinline__ void rv_rows(const Src& src, const RvTeam& t, int rows, const RvVec& v, float* part,
+// `ahead` holds the first 1 + kRvAhead steps' weights when `loaded` is set.  vec(group) is the vector of a group of
+// four rows.
+template <class Src, class Vec>
+__device__ __forceinline__ void rv_rows(const Src& src, const RvTeam& t, int rows, const Vec& vec, float* part,
                                         uint4 (&ahead)[kRvAhead + 1][kRvRows], bool loaded) {
   const int lane = threadIdx.x & 31;
   const int groups = (rows + kRvRows - 1) / kRvRows;
@@ -175,6 +220,7 @@ __device__ __forceinline__ void rv_rows(const Src& src, const RvTeam& t, int row
   for (int s = 0; s < steps; ++s) {
     const int piece = cur.ci * t.threads + t.tid;
     if (piece < t.chunks) {
+      const RvVec v = vec(cur.group);
       const float4 a = reinterpret_cast<const float4*>(v.lo)[piece], b = reinterpret_cast<const float4*>(v.hi)[piece];
 #pragma unroll
       for (int r = 0; r < kRvRows; ++r) {
@@ -204,6 +250,11 @@ __device__ __forceinline__ void rv_rows(const Src& src, const RvTeam& t, int row
     cur.next(t);
   }
 }
+
+struct RvOneVec {
+  RvVec v;
+  __device__ __forceinline__ RvVec operator()(int) const { return v; }
+};
 
 __device__ __forceinline__ float rv_total(const RvTeam& t, const float* part, int row) {
   float s = 0.f;
@@ -252,13 +303,64 @@ __global__ void __launch_bounds__(kRvThreads, 1) rv_dense_kernel(const RvDensePa
       c.next(team);
     }
   }
+  rv_prefetch(p.in);
   pdl_wait();
   rv_stage(p.in, v, red);
   for (int b = r0; b < r1; b += kRvBatchRows) {
     const int rows = min(r1 - b, kRvBatchRows);
-    rv_rows(RvDenseSrc{p.w + b * p.ldw, p.ldw}, team, rows, v, part, ahead, b == r0);
+    rv_rows(RvDenseSrc{p.w + b * p.ldw, p.ldw}, team, rows, RvOneVec{v}, part, ahead, b == r0);
     __syncthreads();
     for (int i = threadIdx.x; i < rows; i += kRvThreads) p.out[b + i] = rv_total(team, part, i) + (p.bias != nullptr ? p.bias[b + i] : 0.f);
+    __syncthreads();
+  }
+}
+
+// ------------------------------------------------------------------ gated halves of one dense feed-forward
+struct RvGatedParams {
+  RvStage in;
+  const __nv_bfloat16* w;  // [2][n][ldw] (gate rows, then up rows)
+  long long ldw;
+  int n;
+  float limit, alpha;
+  float* out;              // [n]
+};
+
+struct RvGatedSrc {        // gate and up rows of a feature as neighbours
+  const __nv_bfloat16* w;
+  long long ldw, half;     // elements between the halves
+  __device__ __forceinline__ uint4 load(int row, int piece) const { return ld_stream(w + (row & 1) * half + (row >> 1) * ldw + piece * 8); }
+};
+
+__global__ void __launch_bounds__(kRvThreads, 1) rv_gated_kernel(const RvGatedParams p) {
+  extern __shared__ __align__(16) float smem[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  const int kp = pad_to(p.in.k, 8);
+  float* part = smem;
+  const RvVec v{smem + kRvBatchRows * kRvWarps, smem + kRvBatchRows * kRvWarps + rv_half_words(kp)};
+  const int f0 = static_cast<int>(static_cast<long long>(p.n) * blockIdx.x / gridDim.x);
+  const int f1 = static_cast<int>(static_cast<long long>(p.n) * (blockIdx.x + 1) / gridDim.x);
+  const RvTeam team(kp / 8);
+  const long long half = p.n * p.ldw;
+  uint4 ahead[kRvAhead + 1][kRvRows];
+  {
+    const RvGatedSrc src{p.w + f0 * p.ldw, p.ldw, half};
+    RvCursor c(team);
+#pragma unroll
+    for (int d = 0; d <= kRvAhead; ++d) {
+      rv_load(src, team, c, min(2 * (f1 - f0), kRvBatchRows), ahead[d]);
+      c.next(team);
+    }
+  }
+  rv_prefetch(p.in);
+  pdl_wait();
+  rv_stage(p.in, v, red);
+  for (int b = f0; b < f1; b += kRvBatchRows / 2) {
+    const int feats = min(f1 - b, kRvBatchRows / 2);
+    rv_rows(RvGatedSrc{p.w + b * p.ldw, p.ldw, half}, team, 2 * feats, RvOneVec{v}, part, ahead, b == f0);
+    __syncthreads();
+    for (int i = threadIdx.x; i < feats; i += kRvThreads)
+      p.out[b + i] = clamped_gate(rv_total(team, part, 2 * i), rv_total(team, part, 2 * i + 1), p.limit, p.alpha);
     __syncthreads();
   }
 }
@@ -297,7 +399,9 @@ __global__ void __launch_bounds__(kRvThreads, 1) rv_gate_up_kernel(const RvGateU
   float* z = v.hi + kp / 2;
   pdl_wait();
   for (int i = threadIdx.x; i < p.n_experts; i += kRvThreads) z[i] = p.logits[i];
-  const RvStage in{p.x, nullptr, nullptr, nullptr, nullptr, 0.f, p.dim};
+  RvStage in{};
+  in.x = p.x;
+  in.k = p.dim;
   rv_stage(in, v, red);
   if (threadIdx.x < 32) {
     select_softmax_warp(z, p.n_experts, p.top, s_ids, s_w);
@@ -325,7 +429,7 @@ __global__ void __launch_bounds__(kRvThreads, 1) rv_gate_up_kernel(const RvGateU
       }
     }
     __syncthreads();
-    rv_rows(RvPtrSrc{s_row}, team, 2 * feats, v, part, ahead, false);
+    rv_rows(RvPtrSrc{s_row}, team, 2 * feats, RvOneVec{v}, part, ahead, false);
     __syncthreads();
     for (int i = threadIdx.x; i < feats; i += kRvThreads) {
       const int f = b + i;
@@ -389,7 +493,7 @@ __global__ void __launch_bounds__(kRvThreads, 1) rv_down_kernel(const RvDownPara
   uint4 ahead[kRvAhead + 1][kRvRows];
   for (int b = r0; b < r1; b += kRvBatchRows) {
     const int rows = min(r1 - b, kRvBatchRows);
-    rv_rows(RvPieceSrc{pieces, b}, team, rows, v, part, ahead, false);
+    rv_rows(RvPieceSrc{pieces, b}, team, rows, RvOneVec{v}, part, ahead, false);
     __syncthreads();
     for (int i = threadIdx.x; i < rows; i += kRvThreads) p.out[b + i] = rv_total(team, part, i);
     __syncthreads();

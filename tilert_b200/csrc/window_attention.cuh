@@ -11,6 +11,9 @@
 //   attn_rows_kernel<T, true>   one token: the preparation, the cache write and the attention in one launch, the
 //                            keys split over CTAs, the last CTA of a head block merging the parts
 //   attn_rows_kernel<T, false>  any number of prepared query rows, f32 arithmetic (the exact mode)
+// The last two read keys and values through strides, so that values may lie inside the keys' rows (a latent cache) or
+// keys may be two pieces, one of them shared by all heads.  The prefill kernel takes an optional sink per head (one more
+// term of the softmax denominator, without key or value) and an optional output gate.
 // Scores, softmax and sums are f32 throughout.
 #pragma once
 
@@ -119,12 +122,16 @@ struct AttnRowsParams {
   QkvShape s;
   QkvPrep p;             // FUSED
   const int* pos;        // position of row 0
-  const void* q;         // !FUSED: [rows, heads, dimp]
+  const void* q;         // !FUSED: row of (head, token) at head * q_head + token * q_token, element type QT
+  long long q_head, q_token;
   void* k_cache;
   void* v_cache;
+  long long v_ld;        // elements between value rows
+  int rows;
+  int parts_only;        // leave every part (n_splits may be 1) for the caller to merge; `out` is not written
   float scale;
   int n_splits;
-  float* part;           // [heads, n_splits, vdimp] and, behind it, [heads, n_splits, 2] (max, sum)
+  float* part;           // [heads, rows, n_splits, vdimp] and, behind it, [heads, rows, n_splits, 2] (max, sum)
   unsigned* counter;     // [head blocks], zero between launches
   void* out;             // [rows, ldo], element type float (FUSED) or T
   long long ldo;
@@ -160,7 +167,7 @@ __device__ __forceinline__ void prefetch_range(const AttnRowsParams& a, int g) {
   }
 }
 
-template <typename T, bool FUSED>
+template <typename T, bool FUSED, typename QT = T>
 __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsParams a) {
   extern __shared__ __align__(16) float smem[];
   __shared__ float red[32];
@@ -182,7 +189,7 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
   const KeyRange range = key_range(pos, s.window, a.n_splits, split);
   const int lo = range.lo, hi = range.hi;
   T* kc = reinterpret_cast<T*>(a.k_cache) + static_cast<long long>(g) * s.ring * s.dimp;
-  T* vc = reinterpret_cast<T*>(a.v_cache) + static_cast<long long>(g) * s.ring * s.vdimp;
+  T* vc = reinterpret_cast<T*>(a.v_cache) + static_cast<long long>(g) * s.ring * a.v_ld;
 
   if (FUSED) {
     const int nq = s.heads * s.dim, nk = s.kv_heads * s.dim;
@@ -201,11 +208,14 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
         act_st(kc + slot * s.dimp + d, row[nq + e] * rk * a.p.k_gain[e]);
       }
       for (int d = tid; d < s.vdim; d += kAttnThreads)
-        act_st(vc + slot * s.vdimp + d, mixed_value(a.p, s, 0, g * s.vdim + d, true));
+        act_st(vc + slot * a.v_ld + d, mixed_value(a.p, s, 0, g * s.vdim + d, true));
     }
   } else {
-    const T* q = reinterpret_cast<const T*>(a.q) + (static_cast<long long>(t) * s.heads + h0) * s.dimp;
-    for (int i = tid; i < kAttnHeads * s.dimp; i += kAttnThreads) qs[i] = i / s.dimp < nh ? act_ld(q + i) * a.scale : 0.f;
+    const QT* q = reinterpret_cast<const QT*>(a.q) + t * a.q_token + h0 * a.q_head;
+    for (int i = tid; i < kAttnHeads * s.dimp; i += kAttnThreads) {
+      const int h = i / s.dimp;
+      qs[i] = h < nh ? act_ld(q + h * a.q_head + (i - h * s.dimp)) * a.scale : 0.f;
+    }
   }
   if (tid < kAttnHeads) {
     s_m[tid] = -INFINITY;
@@ -299,7 +309,7 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
         for (int u = 0; u < kAttnAhead; ++u) {
           const int key = min(k0 + u * key_lanes, cn - 1);
           const int slot = slot0 + key - (slot0 + key >= s.ring ? s.ring : 0);
-          act_ld8(vc + static_cast<long long>(slot) * s.vdimp + vp * 8, f[u]);
+          act_ld8(vc + slot * a.v_ld + vp * 8, f[u]);
         }
 #pragma unroll
         for (int u = 0; u < kAttnAhead; ++u) {
@@ -324,14 +334,15 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
       for (int j = 0; j < 8; ++j) red2[(kl * kAttnHeads + h) * s.vdimp + vp * 8 + j] = acc[h][j];
   }
   __syncthreads();
-  const bool whole = a.n_splits == 1;
-  float* ml = a.part + static_cast<long long>(s.heads) * a.n_splits * s.vdimp;
+  const bool whole = a.n_splits == 1 && !a.parts_only;
+  float* ml = a.part + static_cast<long long>(s.heads) * a.rows * a.n_splits * s.vdimp;
+  auto part_of = [&](int h) { return (static_cast<long long>(h0 + h) * a.rows + t) * a.n_splits; };
   for (int i = tid; i < nh * s.vdimp; i += kAttnThreads) {
     const int h = i / s.vdimp, v = i - h * s.vdimp;
     float o = 0.f;
     for (int k = 0; k < key_lanes; ++k) o += red2[(k * kAttnHeads + h) * s.vdimp + v];
     if (!whole) {
-      a.part[(static_cast<long long>(h0 + h) * a.n_splits + split) * s.vdimp + v] = o;
+      a.part[(part_of(h) + split) * s.vdimp + v] = o;
     } else if (v < s.vdim) {
       const long long dst = t * a.ldo + (h0 + h) * s.vdim + v;
       if (FUSED)
@@ -342,9 +353,10 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
   }
   if (whole) return;
   if (tid < nh) {
-    ml[((h0 + tid) * a.n_splits + split) * 2] = s_m[tid];
-    ml[((h0 + tid) * a.n_splits + split) * 2 + 1] = s_l[tid];
+    ml[(part_of(tid) + split) * 2] = s_m[tid];
+    ml[(part_of(tid) + split) * 2 + 1] = s_l[tid];
   }
+  if (a.parts_only) return;
   // merge by the CTA that finishes its head block last (no CTA waits for another)
   __threadfence();
   __syncthreads();
@@ -359,7 +371,7 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
   // weight of every part, one warp per head: exp(max - overall max), and the overall sum (red2 is free again)
   float* wgt = red2;  // [kAttnHeads][n_splits]
   if (warp < nh) {
-    const float* mh = ml + static_cast<long long>(h0 + warp) * a.n_splits * 2;
+    const float* mh = ml + part_of(warp) * 2;
     float m = -INFINITY, l = 0.f;
     for (int k = lane; k < a.n_splits; k += 32) m = fmaxf(m, __ldcg(mh + 2 * k));
     m = warp_max(m);
@@ -374,7 +386,7 @@ __global__ void __launch_bounds__(kAttnThreads) attn_rows_kernel(const AttnRowsP
   __syncthreads();
   for (int i = tid; i < nh * s.vdim; i += kAttnThreads) {
     const int h = i / s.vdim, v = i - h * s.vdim;
-    const float* src = a.part + static_cast<long long>(h0 + h) * a.n_splits * s.vdimp + v;
+    const float* src = a.part + part_of(h) * s.vdimp + v;
     const float* w = wgt + h * a.n_splits;
     float o = 0.f;
 #pragma unroll 8
@@ -399,9 +411,16 @@ struct AttnPrefillParams {
   const int* pos;        // position of row 0
   int rows;
   const __nv_bfloat16* q;        // [rows, heads, dimp]
-  const __nv_bfloat16* k_cache;  // [kv_heads, ring, dimp]
-  const __nv_bfloat16* v_cache;  // [kv_heads, ring, vdimp]
+  // A key row is dim1 elements of k_cache (head g, row r at g * k_head + r * k_ld), then dimp - dim1 of k2 (row r at
+  // r * k2_ld, the same for all heads); a value row lies at g * v_head + r * v_ld.
+  const __nv_bfloat16* k_cache;
+  const __nv_bfloat16* k2;
+  const __nv_bfloat16* v_cache;
+  long long k_head, k_ld, k2_ld, v_head, v_ld;
+  int dim1;
   float scale;
+  const float* sink;     // optional [heads]
+  HeadGate gate;         // of the output
   __nv_bfloat16* out;    // [rows, ldo]
   long long ldo;
 };
@@ -437,8 +456,8 @@ __global__ void __launch_bounds__(kFaThreads, DV16 <= 8 ? 3 : 1) attn_prefill_ke
   __nv_bfloat16* qs = fsm;
   __nv_bfloat16* ks = qs + kFaRows * qp;
   __nv_bfloat16* vs = ks + 2 * kFaKeys * qp;
-  const __nv_bfloat16* kc = a.k_cache + static_cast<long long>(g) * s.ring * s.dimp;
-  const __nv_bfloat16* vc = a.v_cache + static_cast<long long>(g) * s.ring * s.vdimp;
+  const __nv_bfloat16* kc = a.k_cache + g * a.k_head;
+  const __nv_bfloat16* vc = a.v_cache + g * a.v_head;
   const int lo = s.window > 0 ? max(0, pos0 + t0 - s.window + 1) : 0, hi = pos0 + t0 + nt;  // keys any row sees
 
   const int dch = s.dimp / 8;
@@ -449,18 +468,24 @@ __global__ void __launch_bounds__(kFaThreads, DV16 <= 8 ? 3 : 1) attn_prefill_ke
     const long long row = ok ? static_cast<long long>(t0 + tt) * s.heads + h0 + h : 0;
     cp_async16(qs + r * qp + c * 8, a.q + row * s.dimp + c * 8, ok);
   }
-  auto load_rows = [&](__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int width, int k0) {
-    const int ch = width / 8, slot0 = k0 % s.ring;
+  // rows k0 .. of the keys or values: ch1 pieces of eight from src1, the others from src2
+  auto load_rows = [&](__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src1, long long ld1, int ch1, const __nv_bfloat16* src2,
+                       long long ld2, int ch, int k0) {
+    const int slot0 = k0 % s.ring;
     for (int i = tid; i < kFaKeys * ch; i += kFaThreads) {
       const int r = i / ch, c = i - r * ch;
       const bool ok = k0 + r < hi;
       const long long slot = ok ? slot0 + r - (slot0 + r >= s.ring ? s.ring : 0) : 0;
-      cp_async16(dst + r * pitch + c * 8, src + slot * width + c * 8, ok);
+      cp_async16(dst + r * pitch + c * 8, c < ch1 ? src1 + slot * ld1 + c * 8 : src2 + slot * ld2 + (c - ch1) * 8, ok);
     }
     cp_async_commit();
   };
-  load_rows(ks, qp, kc, s.dimp, lo);
-  load_rows(vs, vpitch, vc, s.vdimp, lo);
+  auto load_keys = [&](int buf, int k0) {
+    load_rows(ks + buf * kFaKeys * qp, qp, kc, a.k_ld, a.dim1 / 8, a.k2, a.k2_ld, s.dimp / 8, k0);
+  };
+  auto load_values = [&](int k0) { load_rows(vs, vpitch, vc, a.v_ld, s.vdimp / 8, vc, a.v_ld, s.vdimp / 8, k0); };
+  load_keys(0, lo);
+  load_values(lo);
 
   float o[DV16 * 2][4];
 #pragma unroll
@@ -482,7 +507,7 @@ __global__ void __launch_bounds__(kFaThreads, DV16 <= 8 ? 3 : 1) attn_prefill_ke
     const bool more = tile + 1 < n_tiles;
     cp_async_wait<1>();  // all but the newest group: this tile's keys (its values are the newest)
     __syncthreads();
-    if (more) load_rows(ks + (buf ^ 1) * kFaKeys * qp, qp, kc, s.dimp, k0 + kFaKeys);
+    if (more) load_keys(buf ^ 1, k0 + kFaKeys);
     const __nv_bfloat16* kt = ks + buf * kFaKeys * qp;
     float sacc[8][4];
 #pragma unroll
@@ -574,7 +599,7 @@ __global__ void __launch_bounds__(kFaThreads, DV16 <= 8 ? 3 : 1) attn_prefill_ke
       }
     }
     __syncthreads();
-    if (more) load_rows(vs, vpitch, vc, s.vdimp, k0 + kFaKeys);
+    if (more) load_values(k0 + kFaKeys);
   }
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
@@ -582,17 +607,28 @@ __global__ void __launch_bounds__(kFaThreads, DV16 <= 8 ? 3 : 1) attn_prefill_ke
     l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
     const int r = warp * 16 + (lane >> 2) + i * 8, tt = r / hpb, h = r - tt * hpb;
     if (tt >= nt || h >= nh) continue;
-    const float inv = 1.f / l[i];
+    float inv = 1.f / l[i];
+    if (a.sink != nullptr) {
+      const float sk = a.sink[h0 + h], top = fmaxf(m[i], sk), e = expf(m[i] - top);
+      inv = e / (l[i] * e + expf(sk - top));
+    }
+    if (a.gate.per_head) inv *= a.gate(t0 + tt, h0 + h, s.vdim, 0);
+    const bool gated = a.gate.z != nullptr && !a.gate.per_head;
     __nv_bfloat16* dst = a.out + static_cast<long long>(t0 + tt) * a.ldo + (h0 + h) * s.vdim;
     const bool pairs = (s.vdim & 1) == 0;
 #pragma unroll
     for (int vb = 0; vb < DV16 * 2; ++vb) {
       const int c = vb * 8 + (lane & 3) * 2;
+      float o0 = o[vb][i * 2] * inv, o1 = o[vb][i * 2 + 1] * inv;
+      if (gated) {
+        if (c < s.vdim) o0 *= a.gate(t0 + tt, h0 + h, s.vdim, c);
+        if (c + 1 < s.vdim) o1 *= a.gate(t0 + tt, h0 + h, s.vdim, c + 1);
+      }
       if (pairs) {
-        if (c < s.vdim) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(o[vb][i * 2] * inv, o[vb][i * 2 + 1] * inv);
+        if (c < s.vdim) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(o0, o1);
       } else {
-        if (c < s.vdim) dst[c] = f2bf(o[vb][i * 2] * inv);
-        if (c + 1 < s.vdim) dst[c + 1] = f2bf(o[vb][i * 2 + 1] * inv);
+        if (c < s.vdim) dst[c] = f2bf(o0);
+        if (c + 1 < s.vdim) dst[c + 1] = f2bf(o1);
       }
     }
   }

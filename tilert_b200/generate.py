@@ -4,7 +4,7 @@ this backend.  No checkpoint or tokenizer ships with the repository, so the runn
 ``prompt_tokens=`` path, generator.py:160,195).
 
     python -m tilert_b200.generate --model toy --use-random-weights --max-new-tokens 32 [--with-mtp]
-    python -m tilert_b200.generate --model ralasun --use-random-weights [--dtype float32]
+    python -m tilert_b200.generate --model ralasun --use-random-weights [--dtype float32]   # likewise --model rozesun
     python -m tilert_b200.generate --model-weights-dir DIR      # the family is chosen by DIR/config.json
 """
 
@@ -21,8 +21,8 @@ from tilert_b200.models import registry
 def parse_args():
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
     ap.add_argument("--model", default="toy", choices=registry.presets(),
-                    help="toy: the 2-layer test model; deepseek_v3_2: the full shape with --layers layers; ralasun: a small "
-                         "model of that design")
+                    help="toy: the 2-layer test model; deepseek_v3_2: the full shape with --layers layers; ralasun, rozesun: "
+                         "a small model of that design")
     ap.add_argument("--dtype", default="bfloat16", help="activation type of a family that runs in more than one")
     ap.add_argument("--layers", type=int, default=2, help="decoder layers of the full-shape model (61 in the real one)")
     ap.add_argument("--use-random-weights", action="store_true")
@@ -50,8 +50,8 @@ def main() -> None:
         raise SystemExit(f"{family.name} runs in {', '.join(family.dtypes)}, not in {args.dtype}")
     if args.with_mtp and family.name != "deepseek_v3_2":
         raise SystemExit(f"{family.name} has no multi-token prediction layer")
-    tilert_b200.load_backend(family.name)
-    tilert_b200.tilert_init(0, family.name)
+    tilert_b200.load_backend(family.backend)
+    tilert_b200.tilert_init(0, family.backend)
     gen = family.generator(weights_dir, args)
     if args.temperature > 0:
         gen.update_sampling_config(args.temperature, args.top_p, args.top_k, args.top_p < 1.0)

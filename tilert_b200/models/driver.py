@@ -3,13 +3,15 @@ next tokens, decode steps replayed from CUDA graphs, prompts in portions, genera
 
 A model supplies ``_step_ops(key)`` -- the operators of one decode step, reading ``self.token`` / ``self.cur_pos`` and
 leaving ``self.logits`` -- and may replace ``prefill`` (by default a prompt goes through the decode step token by
-token)."""
+token).  ``PortionDriver`` is the driver of the models that run a prompt in portions of many tokens."""
 
 from __future__ import annotations
 
 import torch
 
 F32, I32, I64 = torch.float32, torch.int32, torch.int64
+DTYPES = {"bfloat16": torch.bfloat16, "float32": torch.float32}
+MAX_PORTION = 2048  # tokens of a prompt that run at once
 
 
 class SequenceDriver:
@@ -160,3 +162,37 @@ class SequenceDriver:
         return (toks, lgs) if collect_logits else toks
 
     decode_past_last = False  # run the last generated token through the model too
+
+
+class PortionDriver(SequenceDriver):
+    """Prompts in portions (``_prefill_portion``), decode steps whose launch shapes depend on a bound of the keys read."""
+
+    portion: int        # most tokens of a prompt that run at once
+    max_window: int     # most keys any layer attends to
+    # filled by prompts when a caller asks for it: the residual after every layer run, [runs][tokens, dim] f32
+    layer_taps: list[torch.Tensor] | None = None
+
+    def _prefill_portion(self, tokens: list[int], want: list[int], last: bool) -> torch.Tensor:
+        """One portion; f32 logits [len(want), vocab] of the wanted places; with ``last`` also those of the last token
+        in ``self.logits``.  Advances the position."""
+        raise NotImplementedError
+
+    def _graph_key(self, pos: int) -> int:
+        """A bound of the keys any layer attends to: a power of two, constant once every window is full."""
+        n = 256
+        while n < pos + 1 and n < self.max_window:
+            n *= 2
+        return n
+
+    @torch.no_grad()
+    def prefill(self, tokens: list[int], want: list[int] | None = None) -> torch.Tensor:
+        self._check_positions("prefill", self._pos, len(tokens))
+        if len(tokens) == 1:
+            return super().prefill(tokens, want)  # the decode step is the faster form for one token
+        outs = []
+        for lo in range(0, len(tokens), self.portion):
+            part = tokens[lo: lo + self.portion]
+            here = [w - lo for w in (want if want is not None else []) if lo <= w < lo + len(part)]
+            outs.append(self._prefill_portion(part, here, lo + len(part) == len(tokens)))
+        self._choose(self.logits.view(1, -1))
+        return self.logits.view(1, -1).clone() if want is None else torch.cat(outs)

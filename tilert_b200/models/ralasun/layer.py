@@ -12,28 +12,14 @@ itself.  Two forms of the same layer:
 
 from __future__ import annotations
 
-from dataclasses import dataclass
-
 import torch
 
 from tilert_b200 import gqa_ops as ops
 from tilert_b200.gqa_ops import BF16, F32, I32, pad
 from tilert_b200.kv_cache import RingKVCache
 
+from ..blocks import Pending, Scratch, Stream, one_plus, padded_rows
 from .model_args import GATE_ALPHA, LayerArgs, RalasunArgs
-
-
-def padded_rows(w: torch.Tensor, device) -> torch.Tensor:
-    """bf16 [.., n, pad8(k)] on the device, zeros beyond k."""
-    w = w.to(device, BF16)
-    k = w.shape[-1]
-    return w.contiguous() if k % 8 == 0 else torch.nn.functional.pad(w, (0, pad(k) - k)).contiguous()
-
-
-def one_plus(w: torch.Tensor, device) -> torch.Tensor:
-    """f32 gain of a norm whose weight is an offset from one, zeros beyond its length."""
-    g = 1.0 + w.to(device, F32)
-    return torch.nn.functional.pad(g, (0, pad(g.numel()) - g.numel())).contiguous()
 
 
 class LayerWeights:
@@ -87,52 +73,6 @@ class LayerWeights:
             if self.shared_gate_up is not None:
                 n += self.shared_gate_up.numel() + self.shared_down.numel()
         return 2 * n
-
-
-class Scratch:
-    """Named work buffers shared by the layers (they run one after the other).  A buffer is identified by its name
-    and shape, and starts as zeros: what lies beyond a logical length is then zero for good."""
-
-    def __init__(self, device):
-        self.device = torch.device(device)
-        self._bufs: dict = {}
-
-    def get(self, name: str, *shape: int, dtype=F32) -> torch.Tensor:
-        key = (name, shape, dtype)
-        if key not in self._bufs:
-            self._bufs[key] = torch.zeros(*shape, dtype=dtype, device=self.device)
-        return self._bufs[key]
-
-
-@dataclass
-class Pending:
-    """A sublayer output whose norm and residual step the next launch will do."""
-
-    y: torch.Tensor
-    gain: torch.Tensor
-
-
-class Stream:
-    """The residual vector of a one-token step: two buffers, because a launch that advances it reads the old one."""
-
-    def __init__(self, scratch: Scratch, dim: int):
-        self.bufs = [scratch.get("x0", pad(dim)), scratch.get("x1", pad(dim))]
-        self.at = 0
-        self.pending: Pending | None = None
-
-    @property
-    def x(self) -> torch.Tensor:
-        return self.bufs[self.at]
-
-    def dense(self, w, out, n: int, k: int, eps: float, **kw) -> None:
-        """A product of the up-to-date vector; advances the residual when a sublayer output is pending."""
-        if self.pending is None:
-            ops.vec_dense(self.x, w, out, n, k, eps=eps, **kw)
-            return
-        p, nxt = self.pending, self.bufs[self.at ^ 1]
-        ops.vec_dense(self.x, w, out, n, k, y=p.y, gain=p.gain, eps=eps, x_out=nxt, **kw)
-        self.at ^= 1
-        self.pending = None
 
 
 class RalasunLayer:

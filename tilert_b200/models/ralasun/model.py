@@ -6,17 +6,15 @@ from __future__ import annotations
 import torch
 
 from tilert_b200 import gqa_ops as ops
-from tilert_b200.gqa_ops import BF16, F32, I32, I64, pad
+from tilert_b200.gqa_ops import F32, I32, I64, pad
 
-from ..driver import SequenceDriver
-from .layer import LayerWeights, RalasunLayer, Scratch, Stream, one_plus, padded_rows
+from ..blocks import Scratch, Stream, one_plus, padded_rows
+from ..driver import DTYPES, MAX_PORTION, PortionDriver
+from .layer import LayerWeights, RalasunLayer
 from .model_args import RalasunArgs
 
-DTYPES = {"bfloat16": BF16, "float32": F32}
-MAX_PORTION = 2048  # tokens of a prompt that run at once
 
-
-class RalasunModel(SequenceDriver):
+class RalasunModel(PortionDriver):
     backend = "ralasun"
 
     def __init__(self, args: RalasunArgs, sd, device="cuda", dtype: str = "bfloat16", use_graph: bool = True,
@@ -43,8 +41,6 @@ class RalasunModel(SequenceDriver):
             self.layers.append(RalasunLayer(args, li, LayerWeights(args, sd, li, dev), self.scratch, self.portion, self.dtype, dev, v_mode))
         self._init_sequence(dev, args.vocab_size, use_graph)
         self.max_window = max(layer.cache.visible(args.max_seq_len) for layer in self.layers) if self.layers else 1
-        # filled by prefill when a caller asks for it: the residual after every layer, [layers][tokens, dim] f32
-        self.layer_taps: list[torch.Tensor] | None = None
 
     @classmethod
     def from_pretrained(cls, model_dir, device="cuda", dtype: str = "bfloat16", max_seq_len: int | None = None, **kw) -> "RalasunModel":
@@ -61,13 +57,6 @@ class RalasunModel(SequenceDriver):
         return sum(layer.w.weight_bytes(layer.a) for layer in self.layers) + 2 * self.head.numel()
 
     # -- one token --
-    def _graph_key(self, pos: int) -> int:
-        """A bound of the keys any layer attends to: a power of two, constant once every window is full."""
-        n = 256
-        while n < pos + 1 and n < self.max_window:
-            n *= 2
-        return n
-
     def _step_ops(self, length: int) -> None:
         a = self.args
         st = Stream(self.scratch, a.dim)
@@ -83,8 +72,6 @@ class RalasunModel(SequenceDriver):
 
     # -- prompts --
     def _prefill_portion(self, tokens: list[int], want: list[int], last: bool) -> torch.Tensor:
-        """One portion; f32 logits [len(want), vocab] of the wanted places; with ``last`` also those of the last token
-        in ``self.logits``."""
         a, sc, n = self.args, self.scratch, len(tokens)
         ids = torch.tensor(tokens, dtype=I64).to(self.device)
         x, xh = sc.get("x", self.portion, pad(a.dim)), sc.get("xh", self.portion, pad(a.dim), dtype=self.dtype)
@@ -104,16 +91,3 @@ class RalasunModel(SequenceDriver):
         self.cur_pos += n
         self._pos += n
         return out
-
-    @torch.no_grad()
-    def prefill(self, tokens: list[int], want: list[int] | None = None) -> torch.Tensor:
-        self._check_positions("prefill", self._pos, len(tokens))
-        if len(tokens) == 1:
-            return super().prefill(tokens, want)  # the decode step is the faster form for one token
-        outs = []
-        for lo in range(0, len(tokens), self.portion):
-            part = tokens[lo: lo + self.portion]
-            here = [w - lo for w in (want if want is not None else []) if lo <= w < lo + len(part)]
-            outs.append(self._prefill_portion(part, here, lo + len(part) == len(tokens)))
-        self._choose(self.logits.view(1, -1))
-        return self.logits.view(1, -1).clone() if want is None else torch.cat(outs)

@@ -12,7 +12,8 @@ from pathlib import Path
 
 @dataclass(frozen=True)
 class ModelFamily:
-    name: str                          # also the backend's name (tilert_b200.load_backend)
+    name: str
+    backend: str                       # native library with its kernels (tilert_b200.load_backend, build.TARGETS)
     architectures: tuple[str, ...]     # values of "architecture" / "architectures" / "model_type" in config.json
     dtypes: tuple[str, ...]            # activation types the family runs in
     load: Callable                     # (model_dir, device, dtype, max_seq_len) -> a SequenceDriver
@@ -39,6 +40,27 @@ def _ralasun_generator(model_dir, o):
     else:
         model = _ralasun_load(model_dir, "cuda", o.dtype, o.max_seq_len)
     return RalasunGenerator(model, o.max_new_tokens, sampling_seed=o.seed)
+
+
+def _rozesun_load(model_dir, device, dtype, max_seq_len):
+    from .rozesun.model import RozesunModel
+
+    return RozesunModel.from_pretrained(model_dir, device, dtype, max_seq_len)
+
+
+def _rozesun_generator(model_dir, o):
+    from tilert_b200 import synthetic
+
+    from .rozesun.generator import RozesunGenerator
+    from .rozesun.model import RozesunModel
+    from .rozesun.model_args import toy_args
+
+    if model_dir is None:
+        args = toy_args(o.max_seq_len)
+        model = RozesunModel(args, synthetic.random_rozesun_state_dict(args, seed=o.seed), dtype=o.dtype)
+    else:
+        model = _rozesun_load(model_dir, "cuda", o.dtype, o.max_seq_len)
+    return RozesunGenerator(model, o.max_new_tokens, sampling_seed=o.seed)
 
 
 def _dsv32_args(model_dir, max_seq_len):
@@ -81,9 +103,12 @@ def _dsv32_generator(model_dir, o):
 
 
 FAMILIES = (
-    ModelFamily("deepseek_v3_2", ("deepseek_v3_2", "DeepseekV32ForCausalLM", "deepseek_v32"), ("bfloat16",), _dsv32_load, _dsv32_generator,
+    ModelFamily("deepseek_v3_2", "deepseek_v3_2", ("deepseek_v3_2", "DeepseekV32ForCausalLM", "deepseek_v32"), ("bfloat16",), _dsv32_load, _dsv32_generator,
                 presets=("toy", "deepseek_v3_2")),
-    ModelFamily("ralasun", ("Ralasun", "ralasun"), ("bfloat16", "float32"), _ralasun_load, _ralasun_generator, presets=("ralasun",)),
+    ModelFamily("ralasun", "ralasun", ("Ralasun", "ralasun"), ("bfloat16", "float32"), _ralasun_load, _ralasun_generator,
+                presets=("ralasun",)),
+    ModelFamily("rozesun", "ralasun", ("Rozesun", "rozesun"), ("bfloat16", "float32"), _rozesun_load, _rozesun_generator,
+                presets=("rozesun",)),
 )
 
 

@@ -202,3 +202,43 @@ def random_ralasun_state_dict(args, device="cpu", seed: int = 0) -> dict[str, to
             sd |= {f"{p}.mlp.shared.gate": lin(f.shared_ff, d), f"{p}.mlp.shared.up": lin(f.shared_ff, d),
                    f"{p}.mlp.shared.down": lin(d, f.shared_ff)}
     return sd
+
+
+def random_rozesun_state_dict(args, device="cpu", seed: int = 0) -> dict[str, torch.Tensor]:
+    """A random-init Rozesun model under its checkpoint names: as above, with queries and latents large enough for
+    scores that tell keys apart, and sinks of the size of a score."""
+    dev = torch.device(device)
+    gen = torch.Generator(device=dev).manual_seed(seed)
+
+    def rnd(*shape, std=1.0, mean=0.0):
+        return (torch.randn(*shape, generator=gen, dtype=torch.float32, device=dev) * std + mean).to(BF16)
+
+    def lin(n, k):
+        return rnd(n, k, std=k ** -0.5)
+
+    d = args.dim
+    sd = {"embed": rnd(args.vocab_size, d)}
+
+    def norm(name, n):
+        sd.update({name: rnd(n, std=0.2, mean=1.0), f"{name}.b": rnd(n, std=0.2)})
+
+    norm("final.norm", d)
+    if args.loop is not None:
+        sd["loop.step"] = rnd(args.loop.times, d, std=0.5)
+    for i, layer in enumerate(args.layers):
+        m, f = layer.mixer, layer.mlp
+        p = f"l{i}"
+        norm(f"{p}.norm1", d)
+        norm(f"{p}.norm1b", d)
+        sd |= {f"{p}.mix.dq": lin(m.q_rank, d), f"{p}.mix.dq.norm": rnd(m.q_rank, std=0.2, mean=1.6),
+               f"{p}.mix.uq": lin(m.heads * (m.dim + m.rot_dim), m.q_rank), f"{p}.mix.dkv": lin(m.kv_rank + m.rot_dim, d),
+               f"{p}.mix.dkv.norm": rnd(m.kv_rank, std=0.2, mean=1.3), f"{p}.mix.uk": lin(m.heads * m.dim, m.kv_rank),
+               f"{p}.mix.uv": lin(m.heads * m.vdim, m.kv_rank), f"{p}.mix.g": lin(m.heads if m.gate_per_head else m.heads * m.vdim, d),
+               f"{p}.mix.o": lin(d, m.heads * m.vdim)}
+        if m.sink:
+            sd[f"{p}.mix.sink"] = rnd(m.heads, mean=1.5)
+        if f is not None:
+            norm(f"{p}.norm2", d)
+            norm(f"{p}.norm2b", d)
+            sd |= {f"{p}.mlp.gate": lin(f.ff, d), f"{p}.mlp.up": lin(f.ff, d), f"{p}.mlp.down": lin(d, f.ff)}
+    return sd

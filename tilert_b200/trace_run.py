@@ -67,7 +67,7 @@ def main(argv=None) -> int:
         return 3
     from tilert_b200 import build
 
-    build.build(model_type=family.name)  # a fresh checkout has no libraries yet
+    build.build(model_type=family.backend)  # a fresh checkout has no libraries yet
     import tilert_b200 as tb
 
     model = family.load(a.model, "cuda:0", a.dtype, a.max_tokens)
