@@ -724,6 +724,12 @@ def run_c3(args) -> None:
         sys.exit(1)
 
 
+ROZESUN_SIZES = {
+    # name: width, heads (128 + 64 / 128 each), query latent, latent, ff, window of every second layer, cached positions
+    "w2048": (2048, 16, 768, 512, 5632, 1024, 4096),
+    "w4096": (4096, 32, 1536, 512, 11264, 1024, 4096),
+    "w7168": (7168, 64, 1536, 512, 18432, 1024, 4096),
+}
 RALASUN_SIZES = {
     # name: width, query heads, kv heads, experts, top, expert ff, shared ff, window (head sizes 128 / 128), closest model's q_lora
     "w2048": (2048, 16, 4, 64, 6, 1408, 2816, 1024, 768),
@@ -753,6 +759,50 @@ def _graph_us(fn, reps: int) -> float:
     return sorted(ts)[len(ts) // 2]
 
 
+def _model_times(model, toks: list[int], start: int, reps: int) -> tuple[float, float]:
+    """(milliseconds of one portion ``toks`` behind ``start`` cached positions, microseconds of a decode step after it)."""
+    ts = []
+    for i in range(2 + max(reps // 4, 5)):
+        model.reset_sequence()
+        while model._pos < start:
+            model.prefill(toks, [])
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        model.prefill(toks, [])
+        e1.record()
+        torch.cuda.synchronize()
+        ts.append(e0.elapsed_time(e1))
+    prefill_ms = sorted(ts[2:])[len(ts[2:]) // 2]
+    tok = torch.tensor([1], dtype=torch.int64, device="cuda")
+    for _ in range(5):
+        model.forward(tok, model._pos)
+    ts = []
+    for _ in range(reps):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        model.forward(tok, model._pos)
+        e1.record()
+        torch.cuda.synchronize()
+        ts.append(e0.elapsed_time(e1) * 1e3)
+    return prefill_ms, sorted(ts)[len(ts) // 2]
+
+
+def _kernel_table(kernels: dict, layers: list, reps: int):
+    """add(name, fn, bytes, flops): the time of ``fn(layer)``, over all layers' weights in one graph, into ``kernels``."""
+    peak, _ = _peak_gbs()
+
+    def add(name, fn, nbytes=None, nflops=None, layers=layers):
+        us = _graph_us(lambda: [fn(layer) for layer in layers], reps) / len(layers)
+        k = {"us": round(us, 2)}
+        if nbytes:
+            k |= {"bytes": nbytes, "frac_hbm": round(nbytes / us / 1e3 / peak, 3)}
+        if nflops:
+            k |= {"tflops": round(nflops / us / 1e6, 1), "frac_tensor": round(nflops / us / 1e6 / peak_tflops(), 3)}
+        kernels[name] = k
+    return add
+
+
 def _ralasun_arm(size, n_layers: int, portion: int, reps: int) -> dict:
     """Decode and prefill of a stack of equal Ralasun layers, and each of its kernels over the stack's weights."""
     from tilert_b200 import gqa_ops as go
@@ -771,51 +821,17 @@ def _ralasun_arm(size, n_layers: int, portion: int, reps: int) -> dict:
     toks = torch.randint(0, args.vocab_size, (portion,), generator=torch.Generator().manual_seed(1)).tolist()
     start = max(window, portion) // portion * portion  # a full window of cached keys before anything is timed
 
-    # ---- prefill of one portion behind a full window ----
-    ts = []
-    for i in range(2 + max(reps // 4, 5)):
-        model.reset_sequence()
-        while model._pos < start:
-            model.prefill(toks, [])
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        torch.cuda.synchronize()
-        e0.record()
-        model.prefill(toks, [])
-        e1.record()
-        torch.cuda.synchronize()
-        ts.append(e0.elapsed_time(e1))
-    prefill_ms = sorted(ts[2:])[len(ts[2:]) // 2]
+    prefill_ms, step_us = _model_times(model, toks, start, reps)
     flops = portion * n_layers * 2 * (width * (heads * 128 + 2 * kv * 128) + heads * 128 * width + 3 * width * (top * ff + sff) + width * experts) \
         + portion * n_layers * 4 * heads * 128 * window + 2 * width * args.vocab_size
 
-    # ---- decode ----
-    tok = torch.tensor([1], dtype=torch.int64, device="cuda")
-    for _ in range(5):
-        model.forward(tok, model._pos)
-    ts = []
-    for _ in range(reps):
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        e0.record()
-        model.forward(tok, model._pos)
-        e1.record()
-        torch.cuda.synchronize()
-        ts.append(e0.elapsed_time(e1) * 1e3)
-    step_us = sorted(ts)[len(ts) // 2]
     kv_bytes = 2 * kv * 128 * window * 2
     step_bytes = model.weight_bytes() + n_layers * kv_bytes
 
     # ---- the kernels one by one, each over all layers' weights in one graph ----
     peak, _src = _peak_gbs()
     kernels = {}
-
-    def add(name, fn, nbytes=None, nflops=None):
-        us = _graph_us(lambda: [fn(layer) for layer in model.layers], reps) / n_layers
-        k = {"us": round(us, 2)}
-        if nbytes:
-            k |= {"bytes": nbytes, "frac_hbm": round(nbytes / us / 1e3 / peak, 3)}
-        if nflops:
-            k |= {"tflops": round(nflops / us / 1e6, 1), "frac_tensor": round(nflops / us / 1e6 / peak_tflops(), 3)}
-        kernels[name] = k
+    add = _kernel_table(kernels, model.layers, reps)
 
     a, sc, f, eps = args, model.scratch, args.layers[0].mlp, args.eps
     nq, nqkv = heads * 128, heads * 128 + 2 * kv * 128
@@ -985,6 +1001,139 @@ def run_ralasun(args) -> None:
             "ralasun": ours, "closest": {"model": "deepseek_v3_2 layers, FP8 weights, same width / heads / experts", **closest}, "clocks": clocks}), flush=True)
 
 
+def _rozesun_arm(size, n_layers: int, portion: int, reps: int) -> dict:
+    """Decode and prefill of a stack of Rozesun layers, every second one windowed, and each of its kernels over the stack's
+    weights (attention: over the layers of one kind)."""
+    import tilert_b200
+    from tilert_b200 import gqa_ops as go
+    from tilert_b200 import synthetic
+    from tilert_b200.models.blocks import Pending, Stream
+    from tilert_b200.models.rozesun.model import RozesunModel
+    from tilert_b200.models.rozesun.model_args import GATE_ALPHA, LayerArgs, MixerArgs, MlpArgs, RozesunArgs
+
+    width, heads, q_rank, rank, ff, window, ctx = size
+    sizes = dict(heads=heads, dim=128, rot_dim=64, vdim=128, q_rank=q_rank, kv_rank=rank, scale=192 ** -0.5, rot_base=1e4)
+    kinds = (MixerArgs("latent_attention", **sizes), MixerArgs("latent_attention_2", window=window, **sizes))
+    args = RozesunArgs(32768, width, 1e-6, 1.0, tuple(LayerArgs(kinds[i % 2], MlpArgs(ff, 7.0)) for i in range(n_layers)),
+                       max_seq_len=ctx + portion + 4 * reps)
+    model = RozesunModel(args, synthetic.random_rozesun_state_dict(args, "cuda", seed=0), portion=portion)
+    torch.cuda.empty_cache()
+    toks = torch.randint(0, args.vocab_size, (portion,), generator=torch.Generator().manual_seed(1)).tolist()
+    prefill_ms, step_us = _model_times(model, toks, ctx, reps)
+    gates = [m.gate_rows for m in kinds]
+    per_token = [2 * (width * (q_rank + rank + 64 + g + 3 * ff + heads * 128) + q_rank * heads * 192) for g in gates]  # without attention
+    visible = [ctx + portion / 2, window]
+    attn_flops = [2 * portion * heads * v * 320 for v in visible]   # 128 + 64 score products, 128 of the values
+    expand_flops = [2 * n * rank * heads * 256 for n in (ctx + portion, window - 1 + portion)]
+    flops = sum(portion * per_token[i % 2] + attn_flops[i % 2] + expand_flops[i % 2] for i in range(n_layers)) + 2 * width * args.vocab_size
+    cache_bytes = [2 * n * (rank + 64) for n in (ctx + portion, window)]
+    step_bytes = model.weight_bytes() + sum(cache_bytes[i % 2] for i in range(n_layers))
+
+    peak, _src = _peak_gbs()
+    kernels = {}
+    add = _kernel_table(kernels, model.layers, reps)
+    of_kind = [[layer for layer in model.layers if layer.a.mixer is k] for k in kinds]
+    sc, eps, w0 = model.scratch, args.eps, model.layers[0].w
+    row, zmax, nqh = go.latent_row_len(rank, 64), max(layer.z_len for layer in model.layers), heads * 192
+    st = Stream(sc, width)
+    vz, vq, vl, vy = sc.get("b_z", zmax), sc.get("vec_q", nqh), sc.get("vec_lat", heads, row), sc.get("vec_y", width)
+    va, vh, cp = sc.get("vec_att", heads * 128), sc.get("vec_hidden", ff), model.cur_pos
+    vz.normal_(), vq.normal_(), vl.normal_(), vy.normal_(), va.normal_(), vh.normal_()
+
+    def norm_z(layer):
+        st.pending = Pending(vy, layer.w.norm2b)
+        st.dense(layer.w.z, vz, layer.z_len, width, eps, gain2=layer.w.norm1)
+
+    def gated(layer):
+        st.pending = Pending(vy, layer.w.norm1b)
+        st.gated(layer.w.gate_up, vh, ff, width, 7.0, GATE_ALPHA, eps, gain2=layer.w.norm2)
+
+    for i, kind in enumerate(("all keys", "window")):
+        m, n = kinds[i], of_kind[i][0]._splits(1, of_kind[i][0].caches[0].visible(model._pos))
+        part = torch.zeros(heads * n * (rank + 2), device="cuda")
+        add(f"decode input products (+ norms, residual), {kind}", norm_z, 2 * width * of_kind[i][0].z_len, layers=of_kind[i])
+        add(f"decode attention, {kind}", lambda l: go.latent_attn(vl, l.caches[0], 1, m, cp, n, part), cache_bytes[i], layers=of_kind[i])
+        add(f"decode value expansion (+ merge, gate), {kind}", lambda l: go.vec_value(part, l.w.uv, m, n, l.w.sink, vz[l.w.off_g:], m.gate_per_head, va),
+            2 * heads * 128 * rank, layers=of_kind[i])
+    add("decode queries (+ norm)", lambda l: go.vec_dense(vz, l.w.uq, vq, nqh, q_rank, gain2=l.w.q_gain, eps=eps), 2 * nqh * q_rank)
+    add("decode key expansion on queries (+ rotation, cache row)", lambda l: go.vec_absorb(
+        vq, l.w.uk_t, l.a.mixer, l.rope, vz[l.w.off_c:], vz[l.w.off_r:], l.w.c_gain, eps, cp, l.caches[0], vl), 2 * heads * 128 * rank)
+    add("decode output product", lambda l: go.vec_dense(va, l.w.o, vy, width, heads * 128), 2 * heads * 128 * width)
+    add("decode gate/up (+ norms, residual)", gated, 4 * width * ff)
+    add("decode down", lambda l: go.vec_dense(vh, l.w.down, vy, width, ff), 2 * width * ff)
+
+    p, bf = portion, torch.bfloat16
+    model.set_cur_pos(ctx)
+    x, xh, y = sc.get("x", p, width), sc.get("xh", p, width, dtype=bf), sc.get("y", p, width)
+    x.normal_(), xh.normal_(), y.normal_()
+    z, q = sc.flat("z", p, zmax), sc.flat("q", p, nqh)
+    z.normal_(), q.normal_()
+    cq, att, hid = sc.get("cq", p, q_rank, dtype=bf), sc.get("att", p, heads * 128, dtype=bf), sc.get("hid", p, ff, dtype=bf)
+    qe = torch.randn(p, heads, 192, device="cuda").to(bf)
+    zl = model.layers[0].z_len
+    add("prefill input products", lambda l: go.gemm(xh, l.w.z, z, p, zl, width), None, 2 * p * zl * width, layers=of_kind[0])
+    add("prefill latents, cache rows", lambda l: go.latent_tokens(z, l.w.off_c, l.w.off_r, q_rank, l.w.q_gain, l.w.c_gain, eps, p, l.a.mixer, l.rope,
+                                                                  l.caches[0], cp, cq), p * (4 * (q_rank + rank + 64) + 2 * (q_rank + row)))
+    add("prefill queries", lambda l: go.gemm(cq, l.w.uq, q, p, nqh, q_rank), None, 2 * p * nqh * q_rank)
+    add("prefill query rotation", lambda l: go.latent_queries(q, p, l.a.mixer, l.rope, cp, qe), p * nqh * 6)
+    for i, kind in enumerate(("all keys", "window")):
+        m, cached = kinds[i], min(ctx + p, of_kind[i][0].caches[0].ring)
+        kv = torch.zeros(cached, w0.kv.shape[0], dtype=bf, device="cuda")
+        add(f"prefill key/value expansion, {kind}", lambda l: go.gemm(l.caches[0].rows, l.w.kv, kv, cached, kv.shape[1], rank), None,
+            2 * cached * kv.shape[1] * rank, layers=of_kind[i])
+        add(f"prefill attention (+ gate), {kind}", lambda l: go.expanded_attn(qe, kv, l.caches[0], p, m, cp, l.w.sink, z[:, l.w.off_g:], m.gate_per_head, att),
+            None, int(attn_flops[i]), layers=of_kind[i])
+    add("prefill output product", lambda l: go.gemm(att, l.w.o, y, p, width, heads * 128), None, 2 * p * heads * 128 * width)
+    add("prefill norms, residual", lambda l: go.residual_norm(x, xh, l.w.norm1b, eps, width, p, y=y, norm2=l.w.norm2), p * width * 14)
+    add("prefill gate/up", lambda l: go.gemm(xh, l.w.gate_up, hid, p, ff, width, gated=(7.0, GATE_ALPHA)), None, 4 * p * ff * width)
+    add("prefill down", lambda l: go.gemm(hid, l.w.down, y, p, width, ff), None, 2 * p * ff * width)
+    n_few = 16  # a few tokens on many keys: the absorbed form
+    lat = torch.randn(heads * n_few, row, device="cuda")
+    n = of_kind[0][0]._splits(n_few, ctx + p)
+    part = torch.zeros(heads * n_few * n * (rank + 2), device="cuda")
+    add("16 tokens, attention on latents, all keys", lambda l: go.latent_attn(lat, l.caches[0], n_few, kinds[0], cp, n, part), None,
+        2 * heads * n_few * ctx * (2 * rank + 64), layers=of_kind[0])
+    return {"decode_us_per_step": step_us, "decode_tokens_per_s": 1e6 / step_us, "decode_bytes": step_bytes,
+            "decode_frac_hbm": step_bytes / step_us / 1e3 / peak, "decode_us_per_layer": step_us / n_layers,
+            "prefill_ms_per_portion": prefill_ms, "prefill_tokens_per_s": portion / prefill_ms * 1e3,
+            "prefill_tflops": flops / prefill_ms / 1e9, "prefill_frac_tensor": flops / prefill_ms / 1e9 / peak_tflops(),
+            "kernels": kernels, "device_status": tilert_b200.device_status(0, "ralasun")}
+
+
+def run_rozesun(args) -> None:
+    """Layers of the Rozesun design at sizes that resemble a real model's, beside the framework's closest models: Ralasun
+    layers of the same width, head count and feed-forward size (one expert and a shared one of half the size each, so the same
+    weights are read; its attention over the same window and, in a second run, over all keys), and the latent attention of
+    the DeepSeek-V3.2-style layers at the same width and head count.  One JSON line per size; random weights."""
+    import tilert_b200
+
+    for be in ("deepseek_v3_2", "ralasun"):
+        tilert_b200.load_backend(be)
+        tilert_b200.tilert_init(0, be)
+    n_layers, portion, reps = 6, 2048, max(args.steps, 10)
+    for name in args.sizes.split(",") if args.sizes else list(ROZESUN_SIZES):
+        size = ROZESUN_SIZES[name]
+        width, heads, q_rank, rank, ff, window, ctx = size
+        sampler = ClockSampler(0)
+        sampler.start()
+        ours = _rozesun_arm(size, n_layers, portion, reps)
+        clocks = sampler.stop()
+        torch.cuda.empty_cache()
+        closest = {}
+        for label, keys in (("window", window), ("all keys", ctx)):
+            closest[f"ralasun, {label}"] = _ralasun_arm((width, heads, heads // 4, 1, 1, ff // 2, ff // 2, keys, q_rank), n_layers, portion, reps)
+            torch.cuda.empty_cache()
+        closest["deepseek_v3_2"] = _closest_arm((width, heads, heads // 4, 48, 8, 2048, 2048, window, q_rank), n_layers, reps)
+        torch.cuda.empty_cache()
+        print(json.dumps({
+            "metric": "rozesun_decode_tokens_per_s", "value": ours["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": reps,
+            "ms_per_step": ours["decode_us_per_step"] * 1e-3, "higher_is_better": True, "dtype": "bf16 weights, f32 accumulate", "data": "synthetic",
+            "config": {"size": name, "layers": n_layers, "width": width, "heads": heads, "q_rank": q_rank, "kv_rank": rank, "ff": ff, "window": window,
+                       "cached": ctx, "portion": portion, "vocab": 32768, "l2": "one pass reads every layer's own weights: several times the L2",
+                       "peak_hbm_gbs": _peak_gbs()[0], "peak_source": _peak_gbs()[1], "peak_bf16_tflops": peak_tflops()},
+            "rozesun": ours, "closest": closest, "clocks": clocks}), flush=True)
+
+
 def run_profile_gemv(args) -> None:
     """One weight-streaming product alone: N = 7168 rows, K = 32768 (235 MB of FP8 weights, larger
     than L2), a few launches.  Small device footprint, meant to be captured by a profiler."""
@@ -1080,16 +1229,16 @@ def main() -> None:
                     help="short run for a profiler: no clock-sampling loop, no CPU baseline")
     ap.add_argument("--trace-step", action="store_true",
                     help="print the per-launch phase stamps of the streaming products of one step")
-    ap.add_argument("--config", default="c1", choices=["c1", "c2", "c3", "ralasun"],
+    ap.add_argument("--config", default="c1", choices=["c1", "c2", "c3", "ralasun", "rozesun"],
                     help="c1: the headline layer step; c2: whole-model decode (time per output token); c3: long-context "
-                         "indexer + sparse attention stress; ralasun: that design's layers beside the closest model's")
+                         "indexer + sparse attention stress; ralasun, rozesun: that design's layers beside the closest model's")
     ap.add_argument("--ctx", default=None, help="c2: context length(s), comma separated (default 1024); c3: cached keys "
                                                 "(default 131072)")
     ap.add_argument("--chain", default="default", choices=["default", "on", "off", "both"],
                     help="c2: run the layers' products as chained launches, as single launches, or time both")
     ap.add_argument("--with-mtp", action="store_true", help="c2: speculative decoding steps with the prediction layer")
     ap.add_argument("--layers", type=int, default=61, help="c2: decoder layers (61 = the real model; needs 8 GPUs)")
-    ap.add_argument("--sizes", default=None, help="ralasun: comma separated sizes (default: all)")
+    ap.add_argument("--sizes", default=None, help="ralasun, rozesun: comma separated sizes (default: all)")
     ap.add_argument("--gemv-k", type=int, default=32768)
     ap.add_argument("--gemv-packed", action="store_true", help="profile-gemv: activations packed beforehand")
     ap.add_argument("--profile-gemv", action="store_true",
@@ -1105,6 +1254,8 @@ def main() -> None:
         run_c3(args)
     elif args.config == "ralasun" and args.impl == "ours":
         run_ralasun(args)
+    elif args.config == "rozesun" and args.impl == "ours":
+        run_rozesun(args)
     elif args.profile_gemv:
         run_profile_gemv(args)
     elif args.impl == "reference":
