@@ -9,7 +9,7 @@
 //
 // Tensor-core kernel: persistent, warp-specialised, one CTA per SM.  The 128 weight rows of a tile are M (so a TMEM
 // lane is an output feature and a store covers consecutive features), BN token rows are N; K goes by 64.  One thread
-// issues the TMA loads (128-byte swizzle) into a ring of stages, one thread issues the tcgen05.mma, four warps read
+// issues the TMA loads (128-byte swizzle) into a ring of stages, one thread issues the tcgen05.mma, eight warps read
 // the accumulators back; two accumulators alternate so that the epilogue of a tile overlaps the products of the next.
 #pragma once
 
@@ -96,7 +96,8 @@ __device__ __forceinline__ void tile_prefix(const GemmRowsParams& p, int bn, int
 }
 
 // ------------------------------------------------------------------ tensor cores
-constexpr int kTcThreads = 192;  // producer warp, MMA warp, four epilogue warps
+constexpr int kTcEpiWarps = 8;  // two per quarter of the TMEM lanes, each with half of the columns
+constexpr int kTcThreads = 64 + 32 * kTcEpiWarps;  // and a producer warp, an MMA warp
 constexpr int kTcK = 64;
 
 template <int BN, bool GATED>
@@ -150,6 +151,27 @@ __device__ __forceinline__ void tmem_ld16_wait(uint32_t (&r)[16]) {
                : "memory");
 }
 
+// Lane l holds v[t], t = 0 .. 7, of feature l; returns the eight features of the lane's group of eight lanes for token
+// l & 7.  Three exchanges, each between lanes one bit apart, each sending what the partner keeps.
+__device__ __forceinline__ uint4 turn_eight(const float* v, int lane) {
+  const bool b0 = lane & 1, b1 = lane & 2, b2 = lane & 4;
+  uint32_t w[4];         // two features; w[k] of token 2 k + b0
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const float got = __shfl_xor_sync(0xffffffffu, b0 ? v[2 * k] : v[2 * k + 1], 1);
+    w[k] = b0 ? pack_bf16x2(got, v[2 * k + 1]) : pack_bf16x2(v[2 * k], got);
+  }
+  uint32_t lo[2], hi[2];  // four features; of token 4 m + 2 b1 + b0
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const uint32_t got = __shfl_xor_sync(0xffffffffu, b1 ? w[2 * m] : w[2 * m + 1], 2);
+    lo[m] = b1 ? got : w[2 * m];
+    hi[m] = b1 ? w[2 * m + 1] : got;
+  }
+  const uint32_t g0 = __shfl_xor_sync(0xffffffffu, b2 ? lo[0] : lo[1], 4), g1 = __shfl_xor_sync(0xffffffffu, b2 ? hi[0] : hi[1], 4);
+  return b2 ? make_uint4(g0, g1, lo[1], hi[1]) : make_uint4(lo[0], hi[0], g0, g1);
+}
+
 template <int BN, bool GATED>
 __global__ void __launch_bounds__(kTcThreads, 1)
     gemm_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, const GemmRowsParams p) {
@@ -170,7 +192,7 @@ __global__ void __launch_bounds__(kTcThreads, 1)
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&acc_full[i], 1);
-      mbar_init(&acc_empty[i], 4);
+      mbar_init(&acc_empty[i], kTcEpiWarps);
     }
     mbar_init(&drain, 1);
     s_abort = 0;
@@ -259,8 +281,11 @@ __global__ void __launch_bounds__(kTcThreads, 1)
     }
   } else {
     const int quad = warp & 3;  // TMEM lanes this warp may read
+    constexpr int kCols = BN / (kTcEpiWarps / 4);
+    const int c0 = (warp - 2) / 4 * kCols;  // its columns
     const uint32_t lane_off = static_cast<uint32_t>(quad * 32) << 16;
     const bool pairs = p.out_bf16 && (p.n & 1) == 0 && (p.ldo & 1) == 0;
+    const bool eights = p.out_bf16 && (p.n & 7) == 0 && (p.ldo & 7) == 0 && (reinterpret_cast<uintptr_t>(p.out) & 15) == 0;
     uint32_t n_done = 0;
     for (int i = blockIdx.x; i < n_tiles; i += gridDim.x, ++n_done) {
       const TileWalk::Tile t = walk.at(i);
@@ -276,7 +301,7 @@ __global__ void __launch_bounds__(kTcThreads, 1)
       const bool f_ok = f < p.n;
       const float bias = p.bias != nullptr && f_ok ? p.bias[f] : 0.f;
       const uint32_t acc = tmem + buf * S::kAccCols + lane_off;
-      for (int c = 0; c < BN && t.row0 + c < t.row1; c += 16) {
+      for (int c = c0; c < c0 + kCols && t.row0 + c < t.row1; c += 16) {
         float v[16];
         uint32_t r[16];
         tmem_ld16(acc + c, r);
@@ -298,6 +323,15 @@ __global__ void __launch_bounds__(kTcThreads, 1)
 #pragma unroll
           for (int j = 0; j < 16; ++j)
             if (f_ok && j < left) o[j * p.ldo] = v[j];
+        } else if (eights) {
+          // eight lanes turn their eight features of eight tokens over: a lane stores eight features of one token
+          __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(t.row0 + c) * p.ldo + (f & ~7);
+#pragma unroll
+          for (int j = 0; j < 16; j += 8) {
+            const uint4 w = turn_eight(v + j, lane);
+            const int jj = j + (lane & 7);
+            if (f_ok && jj < left) *reinterpret_cast<uint4*>(o + jj * p.ldo) = w;
+          }
         } else if (pairs) {
           // neighbouring lanes exchange one value, so that a lane stores two features of one token
           __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(t.row0 + c) * p.ldo + (f & ~1);
