@@ -69,13 +69,14 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_kernel(const Latent
   }
 
   auto load_keys = [&](int buf, int k0) {
-    const int ch = row / 8, slot0 = k0 % a.ring;
+    const int slot0 = k0 % a.ring;
     __nv_bfloat16* dst = ks + buf * kLaKeys * kp;
-    for (int i = tid; i < kLaKeys * ch; i += kLaThreads) {
-      const int r = i / ch, c = i - r * ch;
+#pragma unroll 2
+    for (int r = warp; r < kLaKeys; r += kLaWarps) {
       const bool ok = k0 + r < hi;
       const long long slot = ok ? slot0 + r - (slot0 + r >= a.ring ? a.ring : 0) : 0;
-      cp_async16(dst + r * kp + c * 8, a.cache + slot * row + c * 8, ok);
+      const __nv_bfloat16* src = a.cache + slot * row;
+      for (int c = lane * 8; c < row; c += 256) cp_async16(dst + r * kp + c, src + c, ok);
     }
     cp_async_commit();
   };

@@ -110,8 +110,11 @@ class RozesunLayer:
         self.ldh = pad(m.dim) + pad(m.rot_dim)
 
     def _splits(self, tokens: int, keys: int) -> int:
-        """Parts of the key range, so that a launch fills the SMs."""
-        return max(1, min(self.sms // ops.latent_blocks(self.a.mixer, tokens, self.dtype), (keys + 63) // 64))
+        """Parts of the key range, of ``per`` tiles of 64 keys each: no more than fill the SMs, and no more than pay (a tile
+        takes about as long as the merge of 24 parts)."""
+        tiles = (keys + 63) // 64
+        least = -(-tiles // max(1, self.sms // ops.latent_blocks(self.a.mixer, tokens, self.dtype)))
+        return min((-(-tiles // per) for per in range(least, least + 4)), key=lambda n: 24 * -(-tiles // n) + n)
 
     # -- one token --
     def decode(self, st: Stream, nr: int, cur_pos: torch.Tensor, length: int) -> None:
